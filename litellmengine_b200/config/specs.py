@@ -24,8 +24,9 @@ class NormSpec:
     kind: str
     eps: float
     weight_name: str = "weight"
-    # kind 'layernorm': (x - mean) * rsqrt(mean((x - mean)^2) + eps) * w, a weight and no bias.
+    # kind 'layernorm': (x - mean) * rsqrt(mean((x - mean)^2) + eps) * w, with `bias` also + b (tensor 'b').
     # kind 'tanh': tanh(alpha * x) * w + b elementwise, no mean and no variance; tensors '<weight>', 'alpha' [], 'b'.
+    bias: bool = False
 
 
 @dataclass(frozen=True)
@@ -41,6 +42,7 @@ class PositionSpec:
     frequencies: with pair(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(pair(fast)), 0),
     hi = min(ceil(pair(slow)), rotary_dim - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency
     is f_i / factor * ramp_i + f_i * (1 - ramp_i); `params` magnitude multiplies cos and sin.
+    kind 'rope_half': the same tables for pairs (i, i + rotary_dim/2), for mixers whose kernels take either layout.
     `params` carries what other kinds need.
     """
     kind: str
@@ -84,6 +86,9 @@ class MixerSpec:
     `head_temperature`: a learned number per query head (tensor 'temp' [heads]) multiplies the scaled score.
     `log_distance_bias`: r1[h] * ln(1 + r2[h] * (i - j)) is taken off the score of query i and key j, with two
     learned numbers per query head (tensors 'r1', 'r2' [heads]); unlike `distance_bias` it has no farthest row.
+    kind 'delta_rule': the gated delta rule with a decay per key channel, short convolutions in front of q, k and v, unit
+    queries and keys, a low-rank sigmoid gate (`num_kv_heads` key heads; `params`: taps, eps of the per-head output norm,
+    decay_rank and gate_rank, None: taken from the stored tensors).
     kind 'latent_attention': softmax attention whose keys and values are made from a cached latent: queries
     through a normed low-rank latent (`params`: q_rank), per token one normed latent of `params` kv_rank entries
     and one rotated key part of `params` rot_dim entries shared by all heads go to the pages; per head the
@@ -118,6 +123,7 @@ class MixerSpec:
     log_distance_bias: bool = False
     keep_first: int = 0                    # with a window: the sequence's first so many keys stay visible to every later query
     softmax_sink: Optional[float] = None   # a score whose exponential joins the softmax's denominator and carries no value
+    learned_sink: bool = False             # the same with a learned score per query head (tensor 'sink' [heads], not scaled)
 
 
 @dataclass(frozen=True)
@@ -126,7 +132,8 @@ class FeedForwardSpec:
     `params` activation names ('silu', 'gelu_tanh': 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))).
     kind 'moe': routed experts; `intermediate_size` is one expert's, `params`: experts, top, groups
     (count, keep) or None, route_scale, limit (the experts' clamp), expert_prefix (expert e's tensors are
-    '<expert_prefix><e>.gate' and so on).
+    '<expert_prefix><e>.gate' and so on), score, correction, router_bias, identity, activation, shared, shared_activation,
+    shared_limit, shared_gate (see `RoutedExperts`).
     `tensor_names`: pairs (the part's own name for a tensor, its name in the model's files)."""
     kind: str
     intermediate_size: int = 0
@@ -152,6 +159,8 @@ class BlockSpec:
     arrangement 'sandwich_norm': h += norm1b(mixer(norm1(h))); h += norm2b(ffn(norm2(h))): a norm in front of each
     sublayer and one on its output (`mixer_post_norm`, `feed_forward_post_norm`, named `mixer_post_norm_name` and
     `feed_forward_post_norm_name`).
+    arrangement 'parallel_pre_norm': h += mixer(u) + ffn(u) with u = norm1(h): one norm that both sublayers read
+    (`feed_forward_norm` None).
     `feed_forward` None: a layer that is its mixer only.
     `connections` = (streams, name of the mixer's connection tensors, name of the feed-forward's): each
     sublayer has tensors `<name>.in` [streams], `<name>.out` [streams], `<name>.mix` [streams, streams]; its
@@ -161,7 +170,7 @@ class BlockSpec:
     mixer: MixerSpec
     feed_forward: Optional[FeedForwardSpec]
     mixer_norm: NormSpec
-    feed_forward_norm: NormSpec
+    feed_forward_norm: Optional[NormSpec]
     weight_prefix: str = ""
     mixer_norm_name: str = "input_layernorm"
     feed_forward_norm_name: str = "post_attention_layernorm"
@@ -182,9 +191,21 @@ class StageSpec:
     A layer named by two stages shares its weights between them, but each stage
     has a cache (or state) of its own, unless `cache_from` names an EARLIER stage
     (by its index in the order) whose cache this stage reads without writing.
+    `starts_pass` = t: in front of this stage the stream is joined with the embedding output as pass t of the model's
+    `rejoin` says.
     """
     block: int
     cache_from: Optional[int] = None
+    starts_pass: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class RejoinSpec:
+    """What happens to the residual stream x in front of a stage with `starts_pass` = t: x <- W [x; x0] + step[t], x0 the
+    embedding output, W [hidden, 2 hidden] the tensor `in_name` (x first), step [passes, hidden] the tensor `step_name`."""
+    passes: int
+    in_name: str = "loop.in"
+    step_name: str = "loop.step"
 
 
 @dataclass(frozen=True)
@@ -204,17 +225,26 @@ class ModelPlan:
     embedding_scale: float = 1.0                          # the token's row is multiplied by this (in 32-bit)
     streams: int = 0                                      # > 0: the layers keep so many copies of the residual stream
                                                           # (equal at the start, summed before the final norm)
+    embedding_norm: Optional[NormSpec] = None             # a norm on the token's row: its output is the embedding output
+    embedding_norm_name: str = "model.embed_norm"
+    rejoin: Optional[RejoinSpec] = None                   # for stages with `starts_pass`
 
     def validate(self) -> None:
         if self.hidden_size <= 0 or self.vocab_size <= 0:
             raise ValueError("hidden_size and vocab_size must be positive")
         if not self.blocks:
             raise ValueError("a model needs at least one layer")
+        if self.embedding_norm is not None and (self.embedding_position is not None or self.streams or self.embedding_scale != 1.0):
+            raise ValueError("a norm on the embedding excludes an added position, a scale and several streams")
+        if self.rejoin is not None and (self.embedding_position is not None or self.streams):
+            raise ValueError("a rejoin with the embedding excludes an added position and several streams")
         if not self.order:
             raise ValueError("the run order is empty")
         for s, st in enumerate(self.order):
             if not 0 <= st.block < len(self.blocks):
                 raise ValueError(f"stage {s} names layer {st.block}, but there are {len(self.blocks)} layers")
+            if st.starts_pass is not None and (self.rejoin is None or self.streams or not 0 <= st.starts_pass < self.rejoin.passes):
+                raise ValueError(f"stage {s} starts pass {st.starts_pass}, which the model's rejoin does not have")
             mixer = self.blocks[st.block].mixer
             conn = self.blocks[st.block].connections
             if (conn[0] if conn else 0) != self.streams:

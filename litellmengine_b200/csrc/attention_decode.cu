@@ -65,7 +65,7 @@ __global__ void __launch_bounds__(AD_THREADS) paged_decode_attention_kernel(
     const int32_t* __restrict__ entry_slot, const int32_t* __restrict__ block_table, int table_stride,
     float* __restrict__ part_acc, float* __restrict__ part_ml, bf16* __restrict__ out, int nq, int nkv,
     int page_size, int window, float scale_log2e, int num_pages, int num_splits, int32_t* __restrict__ status,
-    const float* __restrict__ dist_bias, int dist_len, int keep_first, int has_sink, float sink_log2) {
+    const float* __restrict__ dist_bias, int dist_len, int keep_first, const float* __restrict__ sinks) {
     pdl_begin();
     constexpr int CH = D / 8, KB = D / 16;
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -280,7 +280,7 @@ __global__ void __launch_bounds__(AD_THREADS) paged_decode_attention_kernel(
             L += l_s[w][g] * f;
         }
         if (num_splits == 1) {
-            if (BIAS && has_sink) L += exp2f(sink_log2 - M);        // one more term in the denominator, without a value
+            if (BIAS && sinks) L += exp2f(sinks[h0 + g] * 1.4426950408889634f - M);        // one more term in the denominator, without a value
             out[(static_cast<size_t>(t) * nq + h0 + g) * D + dim] = __float2bfloat16_rn(a / L);
         } else {
             const size_t hrow = static_cast<size_t>(r) * nq + h0 + g;
@@ -299,7 +299,7 @@ __global__ void __launch_bounds__(AD_THREADS) paged_decode_attention_kernel(
 template <int D>
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                             const int32_t* __restrict__ rows, bf16* __restrict__ out, int nq,
-                                            int num_splits, int has_sink, float sink_log2) {
+                                            int num_splits, const float* __restrict__ sinks) {
     pdl_begin();
     const int r = blockIdx.x, h = blockIdx.y;
     const int t = rows ? rows[r] : r;
@@ -318,7 +318,7 @@ __global__ void paged_decode_combine_kernel(const float* __restrict__ part_acc, 
                 L += ls * f;
             }
         }
-        if (has_sink && M != -CUDART_INF_F) L += exp2f(sink_log2 - M);      // a term of the denominator without a value
+        if (sinks && M != -CUDART_INF_F) L += exp2f(sinks[h] * 1.4426950408889634f - M);      // a term of the denominator without a value
         out[(static_cast<size_t>(t) * nq + h) * D + dim] = __float2bfloat16_rn(a / L);
     }
 }
@@ -328,10 +328,9 @@ static int launch_decode(const bf16* q, const bf16* cache, const int32_t* rows, 
                          const int32_t* token_entry, const int32_t* entry_slot, const int32_t* block_table,
                          int table_stride, float* part_acc, float* part_ml, bf16* out, int n_rows, int nq, int nkv,
                          int page_size, int window, float scale, int num_pages, int num_splits, int32_t* status,
-                         const float* dist_bias, int dist_len, int keep_first, int has_sink, float sink_score, cudaStream_t s) {
+                         const float* dist_bias, int dist_len, int keep_first, const float* sinks, cudaStream_t s) {
     const size_t smem = static_cast<size_t>(16 + 2 * AD_STAGES * AD_BN) * D * sizeof(bf16);
-    const bool ext = dist_bias || (keep_first > 0 && window > 0) || has_sink;      // the instantiation that knows them
-    const float sink_log2 = sink_score * 1.4426950408889634f;
+    const bool ext = dist_bias || (keep_first > 0 && window > 0) || sinks;      // the instantiation that knows them
     auto kern = ext ? paged_decode_attention_kernel<D, AD_STAGES, true> : paged_decode_attention_kernel<D, AD_STAGES, false>;
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
@@ -351,7 +350,7 @@ static int launch_decode(const bf16* q, const bf16* cache, const int32_t* rows, 
         launch_pdl(tk, dim3(grid), dim3(AD_THREADS + 32), tsmem, s, *map, q, rows, positions, token_entry, entry_slot, block_table,      \
                                                 table_stride, part_acc, part_ml, out, nq, nkv, page_size, window,    \
                                                 scale * 1.4426950408889634f, num_pages, num_splits, status,          \
-                                                dist_bias, dist_len, keep_first, has_sink, sink_log2);               \
+                                                dist_bias, dist_len, keep_first, sinks);               \
     }
         TMA_GO(3)                                                   // three tiles in shared memory: one read, two in flight
 #undef TMA_GO
@@ -359,13 +358,13 @@ static int launch_decode(const bf16* q, const bf16* cache, const int32_t* rows, 
         launch_pdl(kern, dim3(grid), dim3(AD_THREADS), smem, s, q, cache, rows, positions, token_entry, entry_slot, block_table, table_stride,
                                             part_acc, part_ml, out, nq, nkv, page_size, window,
                                             scale * 1.4426950408889634f, num_pages, num_splits, status, dist_bias, dist_len,
-                                            keep_first, has_sink, sink_log2);
+                                            keep_first, sinks);
     }
     int rc = launch_status();
     if (rc != LLM_OK || num_splits == 1) return rc;
     dim3 cgrid(n_rows, nq);
     launch_pdl((paged_decode_combine_kernel<D>), cgrid, dim3(D <= 64 ? 64 : 128), 0, s, part_acc, part_ml, rows, out, nq, num_splits,
-               has_sink, sink_log2);
+               sinks);
     return launch_status();
 }
 
@@ -387,12 +386,12 @@ extern "C" long long llm_paged_decode_scratch_floats(int n_rows, int nq, int d, 
 // `dist_bias` is float32 [nq, 3], per head a temperature on the scaled score and the two numbers of the bias
 // r1 * ln(1 + r2 * (p - j)) that is taken off it.
 // `keep_first` (with a window): the sequence's first so many keys stay visible; `num_splits` then counts one split
-// more than the window's, which walks them.  `has_sink`: one more term exp(sink_score) in the softmax's denominator.
+// more than the window's, which walks them.  `sinks` (float32 [nq], optional): one more term exp(sinks[head]) in the softmax's denominator.
 extern "C" int llm_paged_attention_decode_ex(
     const void* q, void* out, const void* cache, const int32_t* rows, int n_rows, const int32_t* positions,
     const int32_t* token_entry, const int32_t* entry_slot, const int32_t* block_table, int table_stride, int nq,
     int nkv, int d, int page_size, int window, float scale, int num_pages, int num_splits, float* scratch,
-    int32_t* status, const float* dist_bias, int dist_len, int keep_first, int has_sink, float sink_score,
+    int32_t* status, const float* dist_bias, int dist_len, int keep_first, const float* sinks,
     uintptr_t stream) {
     if (n_rows <= 0) return LLM_OK;
     if (keep_first < 0 || (keep_first > 0 && window > 0 && num_splits < 2)) return LLM_REFUSED_SIZE;
@@ -411,7 +410,7 @@ extern "C" int llm_paged_attention_decode_ex(
     return launch_decode<DD, SS>(static_cast<const bf16*>(q), static_cast<const bf16*>(cache), rows, positions, \
                                  token_entry, entry_slot, block_table, table_stride, part_acc, part_ml,         \
                                  static_cast<bf16*>(out), n_rows, nq, nkv, page_size, window, scale, num_pages, \
-                                 num_splits, status, dist_bias, dist_len, keep_first, has_sink, sink_score, s)
+                                 num_splits, status, dist_bias, dist_len, keep_first, sinks, s)
     if (d == 64) GO(64, 3);
     GO(128, 3);
 #undef GO
@@ -424,7 +423,7 @@ extern "C" int llm_paged_attention_decode_biased(
     int32_t* status, const float* dist_bias, int dist_len, uintptr_t stream) {
     return llm_paged_attention_decode_ex(q, out, cache, rows, n_rows, positions, token_entry, entry_slot, block_table,
                                          table_stride, nq, nkv, d, page_size, window, scale, num_pages, num_splits, scratch,
-                                         status, dist_bias, dist_len, 0, 0, 0.0f, stream);
+                                         status, dist_bias, dist_len, 0, nullptr, stream);
 }
 
 extern "C" int llm_paged_attention_decode(

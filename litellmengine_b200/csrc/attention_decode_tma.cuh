@@ -71,7 +71,7 @@ __global__ void __launch_bounds__(AD_THREADS + 32) paged_decode_attention_tma_ke
     const int32_t* __restrict__ entry_slot, const int32_t* __restrict__ block_table, int table_stride,
     float* __restrict__ part_acc, float* __restrict__ part_ml, bf16* __restrict__ out, int nq, int nkv,
     int page_size, int window, float scale_log2e, int num_pages, int num_splits, int32_t* __restrict__ status,
-    const float* __restrict__ dist_bias, int dist_len, int keep_first, int has_sink, float sink_log2) {
+    const float* __restrict__ dist_bias, int dist_len, int keep_first, const float* __restrict__ sinks) {
     // The wait for the kernel before this one (which writes q and this step's key and value row)
     // comes late: keys and values of earlier steps, the block table and the step's metadata are
     // read first, so the first tiles are already on their way when q arrives.
@@ -318,7 +318,7 @@ __global__ void __launch_bounds__(AD_THREADS + 32) paged_decode_attention_tma_ke
             L += l_s[w][g] * f;
         }
         if (num_splits == 1) {
-            if (BIAS && has_sink) L += exp2f(sink_log2 - M);        // one more term in the denominator, without a value
+            if (BIAS && sinks) L += exp2f(sinks[h0 + g] * 1.4426950408889634f - M);        // one more term in the denominator, without a value
             out[(static_cast<size_t>(t) * nq + h0 + g) * D + dim] = __float2bfloat16_rn(a / L);
         } else {
             const size_t hrow = static_cast<size_t>(r) * nq + h0 + g;

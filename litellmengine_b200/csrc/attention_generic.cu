@@ -38,7 +38,7 @@
 // first part needs no second tensor.  Value widths above 256 take an instantiation with twice the accumulators.
 // `keep_first` (with a window): the first so many keys of the sequence stay visible to every query behind them,
 // at their true positions; the walk is then over the kept keys below the window and the window itself, as one
-// list.  `has_sink`: one more term exp(sink_score) in the softmax's denominator that carries no value.
+// list.  `sinks` (float32 [nq], optional): one more term exp(sinks[head]) in the softmax's denominator that carries no value.
 // With `rows` (int32 [num_tokens]) the kernel works on the listed tokens only (a step's single decoded tokens
 // while its prompt portions take a tensor-core kernel); -1 entries pad the list.
 #include "common.cuh"
@@ -60,7 +60,7 @@ __global__ void paged_attention_generic_kernel(
     long long out_stride, int out_off, int vec, int32_t* __restrict__ status,
     const float* __restrict__ dist_bias, int dist_len, int gate_per_head, const int32_t* __restrict__ rows,
     const float* __restrict__ head_scale, const float* __restrict__ log_r1, const float* __restrict__ log_r2,
-    long long value_row_stride, int keep_first, int has_sink, float sink_score) {
+    long long value_row_stride, int keep_first, const float* sinks) {
     pdl_begin();
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -175,7 +175,7 @@ __global__ void paged_attention_generic_kernel(
         const float mw = merge[w2 * (dv + 2) + dv];
         if (mw != -CUDART_INF_F) l_all += merge[w2 * (dv + 2) + dv + 1] * expf(mw - m_all);
     }
-    if (has_sink) l_all += expf(sink_score - m_all);   // the sink joins the sum; it has no value row (far above every
+    if (sinks) l_all += expf(sinks[h] - m_all);        // the sink joins the sum; it has no value row (far above every
                                                        // score it overflows to infinity and the output to zero: its limit)
     T* orow = out + static_cast<size_t>(t) * out_stride + out_off + static_cast<size_t>(h) * dv;
     const float* grow = gate ? gate + static_cast<size_t>(t) * gate_stride + gate_off +
@@ -203,7 +203,7 @@ extern "C" int llm_paged_attention_generic_kv(
     const float* gate, long long gate_stride, int gate_off, float out_scale, long long out_stride, int out_off,
     int32_t* status, const float* dist_bias, int dist_len, int gate_per_head, const int32_t* rows,
     const float* head_scale, const float* log_r1, const float* log_r2, long long value_row_stride, int keep_first,
-    int has_sink, float sink_score, uintptr_t stream) {
+    const float* sinks, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
     if (keep_first < 0) return LLM_REFUSED_SIZE;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || d > AG_MAX_DK || dv <= 0 || dv > AG_MAX_DV || page_size <= 0)
@@ -226,7 +226,7 @@ extern "C" int llm_paged_attention_generic_kv(
         static_cast<const TC*>(values), key_page_stride, value_page_stride, positions,             \
         token_entry, entry_slot, block_table, table_stride, num_tokens, nq, nkv, d, dv, page_size, \
         window, scale, num_pages, gate, gate_stride, gate_off, out_scale, out_stride, out_off, vec, status, \
-        dist_bias, dist_len, gate_per_head, rows, head_scale, log_r1, log_r2, value_row_stride, keep_first, has_sink, sink_score)
+        dist_bias, dist_len, gate_per_head, rows, head_scale, log_r1, log_r2, value_row_stride, keep_first, sinks)
     if (dtype == LLM_DT_F32 && cache_dtype == LLM_DT_F32) { LAUNCH(float, float); }
     else if (dtype == LLM_DT_BF16 && cache_dtype == LLM_DT_BF16) { LAUNCH(bf16, bf16); }
     else if (dtype == LLM_DT_F32 && cache_dtype == LLM_DT_BF16) { LAUNCH(float, bf16); }
@@ -253,5 +253,5 @@ extern "C" int llm_paged_attention_generic(
                                           cache_dtype, 2 * half, 2 * half, positions, token_entry, entry_slot,
                                           block_table, table_stride, num_tokens, nq, nkv, d, d, page_size, window,
                                           scale, num_pages, nullptr, 0, 0, 1.0f, static_cast<long long>(nq) * d, 0,
-                                          status, nullptr, 0, 0, nullptr, nullptr, nullptr, nullptr, 0, 0, 0, 0.0f, stream);
+                                          status, nullptr, 0, 0, nullptr, nullptr, nullptr, nullptr, 0, 0, nullptr, stream);
 }

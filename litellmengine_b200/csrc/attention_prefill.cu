@@ -66,7 +66,7 @@ __global__ void __launch_bounds__(AP_THREADS) paged_prefill_attention_kernel(
     const int32_t* __restrict__ block_table, int table_stride, int nq, int nkv, int page_size, int window,
     float scale_log2e, int num_pages, int32_t* __restrict__ status,
     const float* __restrict__ dist_bias, int dist_len, const float* __restrict__ head_gate, long long gate_stride,
-    int gate_off, float out_scale, long long out_stride, int out_off, int keep_first, int has_sink, float sink_log2) {
+    int gate_off, float out_scale, long long out_stride, int out_off, int keep_first, const float* __restrict__ sinks) {
     pdl_begin();
     constexpr int CH = D / 8;                     // 16-byte chunks per row
     constexpr int KB = D / 16;                    // k-blocks of the first product
@@ -281,7 +281,8 @@ __global__ void __launch_bounds__(AP_THREADS) paged_prefill_attention_kernel(
     }
     cp_async_wait_all();
 
-    if (EXT && has_sink) {                            // one more term in the denominator, without a value
+    if (EXT && sinks) {                            // one more term in the denominator, without a value
+        const float sink_log2 = sinks[h] * 1.4426950408889634f;
         if (m0 != -CUDART_INF_F) l0 += exp2f(sink_log2 - m0);
         if (m1 != -CUDART_INF_F) l1 += exp2f(sink_log2 - m1);
     }
@@ -308,7 +309,7 @@ extern "C" int llm_paged_attention_prefill_ex(
     const int32_t* entry_q_start, const int32_t* entry_q_len, const int32_t* entry_kv_len,
     const int32_t* block_table, int table_stride, int nq, int nkv, int d, int page_size, int window, float scale,
     int num_pages, int32_t* status, const float* dist_bias, int dist_len, const float* head_gate, long long gate_stride,
-    int gate_off, float out_scale, long long out_stride, int out_off, int keep_first, int has_sink, float sink_score,
+    int gate_off, float out_scale, long long out_stride, int out_off, int keep_first, const float* sinks,
     uintptr_t stream);
 
 // q, out: bfloat16 [T, nq*d]; cache: bfloat16 [pages, 2, nkv, page_size, d];
@@ -321,7 +322,7 @@ extern "C" int llm_paged_attention_prefill(
     int num_pages, int32_t* status, uintptr_t stream) {
     return llm_paged_attention_prefill_ex(q, out, cache, tiles, n_tiles, entry_slot, entry_q_start, entry_q_len, entry_kv_len,
                                           block_table, table_stride, nq, nkv, d, page_size, window, scale, num_pages, status,
-                                          nullptr, 0, nullptr, 0, 0, 1.0f, static_cast<long long>(nq) * d, 0, 0, 0, 0.0f, stream);
+                                          nullptr, 0, nullptr, 0, 0, 1.0f, static_cast<long long>(nq) * d, 0, 0, nullptr, stream);
 }
 
 // The same with what other attention layers add: `dist_bias` float32 [nq, dist_len], a learned bias by distance in
@@ -329,14 +330,14 @@ extern "C" int llm_paged_attention_prefill(
 // query i and key j (dist_len == -1: `dist_bias` is float32 [nq, 3] = a temperature on the scaled score and the two
 // numbers of the bias r1 * ln(1 + r2 * (i - j)) that is taken off it, per head); `head_gate` float32, one value per (token, head) at [token * gate_stride + gate_off + head],
 // whose sigmoid multiplies the head's output; `out_scale`; the output row as a column range of a wider buffer;
-// `keep_first`: with a window, the sequence's first so many keys stay visible to every later query; `has_sink`: one
-// more term exp(sink_score) in the softmax's denominator that carries no value.
+// `keep_first`: with a window, the sequence's first so many keys stay visible to every later query; `sinks` (float32 [nq],
+// optional): one more term exp(sinks[head]) in the softmax's denominator that carries no value.
 extern "C" int llm_paged_attention_prefill_ex(
     const void* q, void* out, const void* cache, const int32_t* tiles, int n_tiles, const int32_t* entry_slot,
     const int32_t* entry_q_start, const int32_t* entry_q_len, const int32_t* entry_kv_len,
     const int32_t* block_table, int table_stride, int nq, int nkv, int d, int page_size, int window, float scale,
     int num_pages, int32_t* status, const float* dist_bias, int dist_len, const float* head_gate, long long gate_stride,
-    int gate_off, float out_scale, long long out_stride, int out_off, int keep_first, int has_sink, float sink_score,
+    int gate_off, float out_scale, long long out_stride, int out_off, int keep_first, const float* sinks,
     uintptr_t stream) {
     if (n_tiles <= 0) return LLM_OK;
     if (keep_first < 0) return LLM_REFUSED_SIZE;
@@ -348,7 +349,7 @@ extern "C" int llm_paged_attention_prefill_ex(
     dim3 grid(nq, n_tiles);
     const float scale_log2e = scale * 1.4426950408889634f;
     const bool ext = dist_bias || head_gate || out_scale != 1.0f || out_off != 0 || out_stride != static_cast<long long>(nq) * d ||
-                     (keep_first > 0 && window > 0) || has_sink;
+                     (keep_first > 0 && window > 0) || sinks;
 #define LAUNCH(DD)                                                                                             \
     {                                                                                                          \
         auto kern = ext ? paged_prefill_attention_kernel<DD, true> : paged_prefill_attention_kernel<DD, false>;    \
@@ -360,7 +361,7 @@ extern "C" int llm_paged_attention_prefill_ex(
                                             entry_q_len, entry_kv_len, block_table, table_stride, nq, nkv,     \
                                             page_size, window, scale_log2e, num_pages, status, dist_bias,      \
                                             dist_len, head_gate, gate_stride, gate_off, out_scale, out_stride, out_off, \
-                                            keep_first, has_sink, sink_score * 1.4426950408889634f); \
+                                            keep_first, sinks); \
     }
     if (d == 64) LAUNCH(64) else LAUNCH(128)
 #undef LAUNCH

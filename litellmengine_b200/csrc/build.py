@@ -33,6 +33,7 @@ FAMILIES: Dict[str, List[str]] = {
     "attention_generic": ["attention_generic.cu"],
     "attention_prepare": ["attention_prepare.cu"],
     "linear_attention": ["linear_attention.cu"],
+    "delta_rule": ["delta_rule.cu"],
     "streams": ["streams.cu"],
     "conv_norm": ["conv_norm.cu"],
     "latent_attention": ["latent_attention.cu"],

@@ -114,6 +114,90 @@ extern "C" int llm_embedding_sinusoid(const int32_t* ids, const void* table, int
     return launch_status();
 }
 
+// The gather with the model's norm behind it: out[t, :] = norm(table[id, :]) * w (+ b), layer norm (`center`: mean, then
+// the mean of the squared deviations) or RMS norm, in 32-bit; `copy` (optional) receives the same row in the compute
+// dtype.  One block per token; the row waits in shared memory between the passes.
+template <typename T, typename TC>
+__global__ void embedding_norm_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table, const float* __restrict__ w,
+                                      const float* __restrict__ b, float eps, int center, float* __restrict__ out,
+                                      TC* __restrict__ copy, int hidden, int vocab, int32_t* __restrict__ status,
+                                      const int32_t* __restrict__ feedback, int feedback_len) {
+    pdl_begin();
+    extern __shared__ __align__(16) float row_s[];
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    int id = ids[t];
+    if (id < 0 && feedback != nullptr && -1 - id < feedback_len) id = feedback[-1 - id];
+    const bool bad = id < 0 || id >= vocab;
+    if (bad && threadIdx.x == 0 && atomicCAS(status, 0, 1) == 0) status[1] = t;
+    const T* row = table + static_cast<size_t>(bad ? 0 : id) * hidden;
+    float sum = 0.0f;
+    if ((hidden & 7) == 0) {
+        for (int h = threadIdx.x * 8; h < hidden; h += blockDim.x * 8) {
+            float v[8];
+            load8(row + h, v);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                v[i] = bad ? 0.0f : v[i];
+                row_s[h + i] = v[i];
+                sum += v[i];
+            }
+        }
+    } else {
+        for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+            const float v = bad ? 0.0f : to_f32(row[h]);
+            row_s[h] = v;
+            sum += v;
+        }
+    }
+    float mean = 0.0f;
+    if (center) mean = block_sum(sum, scratch) / static_cast<float>(hidden);
+    __syncthreads();
+    float ss = 0.0f;
+    for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+        const float d = row_s[h] - mean;
+        ss += d * d;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps);
+    float* o = out + static_cast<size_t>(t) * hidden;
+    TC* c = copy ? copy + static_cast<size_t>(t) * hidden : nullptr;
+    for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+        const float v = (row_s[h] - mean) * inv * w[h] + (b ? b[h] : 0.0f);
+        o[h] = v;
+        if (c) c[h] = from_f32<TC>(v);
+    }
+}
+
+extern "C" int llm_embedding_norm(const int32_t* ids, const void* table, int table_dtype, const float* w, const float* b, float eps,
+                                  int center, float* out, void* copy, int copy_dtype, int num_tokens, int hidden, int vocab,
+                                  int32_t* status, const int32_t* feedback, int feedback_len, uintptr_t stream) {
+    if (num_tokens <= 0) return LLM_OK;
+    if (hidden <= 0 || vocab <= 0 || hidden > 48 * 1024) return LLM_REFUSED_SIZE;
+    if ((hidden & 7) == 0 && !aligned16(table)) return LLM_REFUSED_ALIGN;
+    const int threads = hidden >= 2048 ? 256 : 128;
+    const size_t smem = static_cast<size_t>(hidden) * sizeof(float);
+    cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define LAUNCH(T, TC)                                                                                          \
+    do {                                                                                                       \
+        auto kern = embedding_norm_kernel<T, TC>;                                                              \
+        if (smem > 47 * 1024) {                                                                                \
+            const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,      \
+                                                       static_cast<int>(smem));                                \
+            if (e != cudaSuccess) return static_cast<int>(e);                                                  \
+        }                                                                                                      \
+        launch_pdl(kern, dim3(num_tokens), dim3(threads), smem, s, ids, static_cast<const T*>(table), w, b,    \
+                   eps, center, out, static_cast<TC*>(copy), hidden, vocab, status, feedback, feedback_len);   \
+    } while (0)
+    if (!copy) copy_dtype = LLM_DT_F32;
+    if (table_dtype == LLM_DT_F32 && copy_dtype == LLM_DT_F32) LAUNCH(float, float);
+    else if (table_dtype == LLM_DT_F32 && copy_dtype == LLM_DT_BF16) LAUNCH(float, bf16);
+    else if (table_dtype == LLM_DT_BF16 && copy_dtype == LLM_DT_F32) LAUNCH(bf16, float);
+    else if (table_dtype == LLM_DT_BF16 && copy_dtype == LLM_DT_BF16) LAUNCH(bf16, bf16);
+    else return LLM_REFUSED_DTYPE;
+#undef LAUNCH
+    return launch_status();
+}
+
 // dst[index[i]] = value[i] for i < *count (count lives on the device so that a captured
 // graph can replay with a different number of updates; a null count means max_count).  An index outside [0, dst_len)
 // is skipped and recorded in status.

@@ -14,6 +14,9 @@
 //                    expert at all: a token that picks one gets its own input back times the weight.  Those
 //                    have no column in the dense row (it has E - identity columns), their place in the lists
 //                    holds id -1 and weight 0, and the sum of their weights goes to `idw` [tokens].
+//                    `bias` (float32 [router outputs], optional) joins the logits themselves, before any score.
+//                    `shared_w` (float32 [W], optional): one more row, whose product's sigmoid goes to `share` [tokens]
+//                    (the weight of an expert that every token runs).
 //                    The experts' activation: g = min(gate, limit), u = clamp(up, -limit, limit),
 //                    w * g * sigmoid(alpha g) * (u + up_shift); limit = infinity, alpha = 1, up_shift = 0 is
 //                    the plain silu(gate) * up.
@@ -32,7 +35,8 @@ template <typename TX>
 __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restrict__ wr, float* __restrict__ dense,
                                  int32_t* __restrict__ ids, float* __restrict__ weights, int num_tokens, int W, int E,
                                  int top, int groups, int keep, float route_scale, int vec, int softmax,
-                                 const float* __restrict__ correction, int identity, float* __restrict__ idw) {
+                                 const float* __restrict__ correction, int identity, float* __restrict__ idw,
+                                 const float* __restrict__ bias, const float* __restrict__ shared_w, float* __restrict__ share) {
     pdl_begin();
     extern __shared__ float smem[];
     const int G = groups > 0 ? groups : 1;
@@ -54,8 +58,9 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
         for (int i = tid; i < nt * W; i += blockDim.x) xs[i] = to_f32(x[t0 * W + i]);
     }
     __syncthreads();
-    for (int e = warp; e < E; e += MOE_ROUTE_THREADS / 32) {       // a warp an expert: its row against the block's tokens
-        const float* w = wr + static_cast<size_t>(e) * W;
+    const int rows = E + (shared_w ? 1 : 0);
+    for (int e = warp; e < rows; e += MOE_ROUTE_THREADS / 32) {    // a warp an expert: its row against the block's tokens
+        const float* w = e < E ? wr + static_cast<size_t>(e) * W : shared_w;
         float dot[MOE_ROUTE_TOKENS];
 #pragma unroll
         for (int k = 0; k < MOE_ROUTE_TOKENS; ++k) dot[k] = 0.0f;
@@ -78,7 +83,12 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
         }
 #pragma unroll
         for (int k = 0; k < MOE_ROUTE_TOKENS; ++k) {
-            const float d = warp_sum(dot[k]);
+            float d = warp_sum(dot[k]);
+            if (e == E) {
+                if (lane == 0 && k < nt) share[t0 + k] = 1.0f / (1.0f + expf(-d));
+                continue;
+            }
+            if (bias) d += bias[e];
             if (lane == 0 && k < nt) score[k * E + e] = softmax ? d : 1.0f / (1.0f + expf(-d));
         }
     }
@@ -163,7 +173,8 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
 
 extern "C" int llm_moe_route(const void* x, int x_dtype, const float* wr, float* dense, int32_t* ids, float* weights,
                              int num_tokens, int W, int E, int top, int groups, int keep, float route_scale,
-                             int softmax, const float* correction, int identity, float* idw, uintptr_t stream) {
+                             int softmax, const float* correction, int identity, float* idw, const float* bias,
+                             const float* shared_w, float* share, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
     if (identity < 0 || identity >= E || (identity > 0 && !idw)) return LLM_REFUSED_SIZE;
     if (W <= 0 || E <= 0 || top <= 0 || top > E || top > 64 || groups < 0) return LLM_REFUSED_SIZE;
@@ -172,7 +183,8 @@ extern "C" int llm_moe_route(const void* x, int x_dtype, const float* wr, float*
     if (smem > 200 * 1024) return LLM_REFUSED_SIZE;
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
     const dim3 grid((num_tokens + MOE_ROUTE_TOKENS - 1) / MOE_ROUTE_TOKENS);
-    const int vec = W % 8 == 0 && aligned16(x) && aligned16(wr);
+    if (shared_w && !share) return LLM_REFUSED_SIZE;
+    const int vec = W % 8 == 0 && aligned16(x) && aligned16(wr) && (!shared_w || aligned16(shared_w));
 #define LAUNCH(TX)                                                                                                  \
     do {                                                                                                            \
         auto kern = moe_route_kernel<TX>;                                                                           \
@@ -182,7 +194,8 @@ extern "C" int llm_moe_route(const void* x, int x_dtype, const float* wr, float*
             if (e != cudaSuccess) return static_cast<int>(e);                                                       \
         }                                                                                                           \
         launch_pdl(kern, grid, dim3(MOE_ROUTE_THREADS), smem, s, static_cast<const TX*>(x), wr, dense, ids, weights,  \
-                   num_tokens, W, E, top, groups, keep, route_scale, vec, softmax, correction, identity, idw);      \
+                   num_tokens, W, E, top, groups, keep, route_scale, vec, softmax, correction, identity, idw, bias, \
+                   shared_w, share);                                                                                \
     } while (0)
     if (x_dtype == LLM_DT_F32) LAUNCH(float);
     else if (x_dtype == LLM_DT_BF16) LAUNCH(bf16);
@@ -205,21 +218,29 @@ __device__ __forceinline__ void moe_store4(bf16* p, const float (&v)[4]) {
     *reinterpret_cast<uint2*>(p) = raw;
 }
 
-// One block row per (token, expert): the token's weight for the expert is read once; a thread makes VEC
+// One block row per (token, expert), the shared expert (when `ffs` > 0) behind the routed ones: its gate and up values
+// follow the routed experts' in a row of `gu`, its activations follow theirs in a row of `act`, its size and limit are
+// its own and its weight is `share` [token] (null: one).  The token's weight for the expert is read once; a thread makes VEC
 // neighbouring features (VEC = 4: sixteen-byte loads of the gate and up values, which are only touched
 // for experts that were chosen; the others' columns are zeroed).
 template <typename TO, int VEC>
 __global__ void moe_act_kernel(const float* __restrict__ gu, int parts, long long part_stride,
-                               const float* __restrict__ dense, TO* __restrict__ act, int E, int ff, float limit,
-                               float alpha, float shift) {
+                               const float* __restrict__ dense, TO* __restrict__ act, int E, int ff_routed, float limit,
+                               float alpha, float shift, int ffs, float limit_s, const float* __restrict__ share) {
     pdl_begin();
-    const long long pair = blockIdx.x;                  // token * E + expert
+    const int slots = E + (ffs > 0 ? 1 : 0);
+    const long long t = blockIdx.x / slots;
+    const int e = static_cast<int>(blockIdx.x - t * slots);
+    const bool routed = e < E;
+    const int ff = routed ? ff_routed : ffs;
     const int f = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
     if (f >= ff) return;
-    const float w = dense[pair];
+    const long long width = static_cast<long long>(E) * ff_routed + ffs, first = static_cast<long long>(e) * ff_routed;
+    const float w = routed ? dense[t * E + e] : (share ? share[t] : 1.0f);
+    if (!routed) limit = limit_s;
     float out[4] = {0.0f, 0.0f, 0.0f, 0.0f};
     if (w != 0.0f) {
-        const float* p = gu + pair * 2 * ff;
+        const float* p = gu + 2 * (t * width + first);
         float g[4] = {0.0f, 0.0f, 0.0f, 0.0f}, u[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         for (int k = 0; k < parts; ++k) {                   // the product may come as its k-splits
             if (VEC == 4) {
@@ -235,27 +256,29 @@ __global__ void moe_act_kernel(const float* __restrict__ gu, int parts, long lon
 #pragma unroll
         for (int c = 0; c < VEC; ++c) out[c] = w * moe_activate(g[c], u[c], limit, alpha, shift);
     }
-    TO* o = act + pair * ff + f;
+    TO* o = act + t * width + first + f;
     if (VEC == 4) moe_store4(o, out);
     else o[0] = from_f32<TO>(out[0]);
 }
 
 extern "C" int llm_moe_act(const float* gu, int parts, long long part_stride, const float* dense, void* act,
                            int act_dtype, int num_tokens, int E, int ff, float limit, float alpha, float shift,
-                           uintptr_t stream) {
+                           int ffs, float limit_s, const float* share, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
-    if (E <= 0 || ff <= 0 || !(limit > 0.0f)) return LLM_REFUSED_SIZE;
-    const long long pairs = static_cast<long long>(num_tokens) * E;
+    // E = 0: a shared expert alone
+    if (E < 0 || ff < 0 || ffs < 0 || (E > 0 && (ff <= 0 || !(limit > 0.0f) || !dense)) || (ffs > 0 && !(limit_s > 0.0f)) || E + ffs <= 0)
+        return LLM_REFUSED_SIZE;
+    const long long pairs = static_cast<long long>(num_tokens) * (E + (ffs > 0 ? 1 : 0));
     if (pairs > 0x7fffffffLL) return LLM_REFUSED_SIZE;
     if (parts < 1) parts = 1;
-    const bool vec = ff % 4 == 0 && aligned16(gu) && aligned16(act) && part_stride % 4 == 0;
-    const int per_block = 128 * (vec ? 4 : 1);
-    const dim3 grid(static_cast<unsigned>(pairs), (ff + per_block - 1) / per_block);
+    const bool vec = ff % 4 == 0 && ffs % 4 == 0 && aligned16(gu) && aligned16(act) && part_stride % 4 == 0;
+    const int per_block = 128 * (vec ? 4 : 1), widest = ff > ffs ? ff : ffs;
+    const dim3 grid(static_cast<unsigned>(pairs), (widest + per_block - 1) / per_block);
     if (grid.y > 65535) return LLM_REFUSED_SIZE;
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define LAUNCH(TO, V)                                                                                          \
     launch_pdl((moe_act_kernel<TO, V>), grid, dim3(128), 0, s, gu, parts, part_stride, dense, static_cast<TO*>(act), E, ff, \
-               limit, alpha, shift)
+               limit, alpha, shift, ffs, limit_s, share)
     if (act_dtype == LLM_DT_F32) { if (vec) LAUNCH(float, 4); else LAUNCH(float, 1); }
     else if (act_dtype == LLM_DT_BF16) { if (vec) LAUNCH(bf16, 4); else LAUNCH(bf16, 1); }
     else return LLM_REFUSED_DTYPE;
@@ -270,7 +293,7 @@ extern "C" int llm_moe_act(const float* gu, int parts, long long part_stride, co
 // memory (32-bit accumulation), so the chosen experts' bytes bound them.
 //   moe_gate_up_sparse_kernel   act[pair, f] = w * g * sigmoid(alpha g) * (u + 1) for pair = (token, k-th choice)
 //   moe_down_sparse_kernel      out[token, n] = sum over the token's choices of W_down[e][n, :] . act[pair, :]
-// Weights: `w_gate_up` [E * 2 * ff, W] (per expert ff gate rows, then ff up rows) and `w_down` [W, E * ff].
+// Weights: `w_gate_up` [E * 2 * ff, W] (per expert ff gate rows, then ff up rows) and `w_down` [W, E * ff] (rows `down_stride` elements apart).
 #define MOE_SPARSE_WARPS 8
 #define MOE_SPARSE_FEATURES 8
 
@@ -366,7 +389,7 @@ __global__ void moe_gate_up_sparse_kernel(const TX* __restrict__ x, const TW* __
 template <typename TA, typename TW>
 __global__ void moe_down_sparse_kernel(const TA* __restrict__ act, const TW* __restrict__ wd,
                                        const int32_t* __restrict__ ids, float* __restrict__ out, int W, int ff, int top,
-                                       int E, int vec) {
+                                       long long ld, int vec) {
     pdl_begin();
     extern __shared__ __align__(16) float as[];        // [top * ff]
     const int t = blockIdx.x;
@@ -375,7 +398,7 @@ __global__ void moe_down_sparse_kernel(const TA* __restrict__ act, const TW* __r
     __syncthreads();
     const int n0 = blockIdx.y * MOE_SPARSE_FEATURES;
     for (int n = n0 + warp; n < min(W, n0 + MOE_SPARSE_FEATURES); n += MOE_SPARSE_WARPS) {
-        const TW* row = wd + static_cast<size_t>(n) * E * ff;
+        const TW* row = wd + static_cast<size_t>(n) * ld;
         float acc = 0.0f;
         for (int k = 0; k < top; ++k) {
             const int e = ids[t * top + k];
@@ -387,13 +410,13 @@ __global__ void moe_down_sparse_kernel(const TA* __restrict__ act, const TW* __r
 
 extern "C" int llm_moe_sparse(const void* x, int x_dtype, const void* wgu, const void* wd, int w_dtype, const int32_t* ids,
                               const float* weights, void* act, float* out, int num_tokens, int W, int ff, int E, int top,
-                              float limit, float alpha, float shift, uintptr_t stream) {
+                              float limit, float alpha, float shift, long long down_stride, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
-    if (W <= 0 || ff <= 0 || E <= 0 || top <= 0 || !(limit > 0.0f)) return LLM_REFUSED_SIZE;
+    if (W <= 0 || ff <= 0 || E <= 0 || top <= 0 || !(limit > 0.0f) || down_stride < static_cast<long long>(E) * ff) return LLM_REFUSED_SIZE;
     const size_t smem_a = static_cast<size_t>(W) * sizeof(float), smem_b = static_cast<size_t>(top) * ff * sizeof(float);
     if (smem_a > 48 * 1024 || smem_b > 48 * 1024) return LLM_REFUSED_SIZE;
     if (x_dtype != w_dtype) return LLM_REFUSED_DTYPE;       // the activations between the two kernels take the tokens' dtype
-    const int vec = W % 8 == 0 && ff % 8 == 0 && aligned16(wgu) && aligned16(wd);
+    const int vec = W % 8 == 0 && ff % 8 == 0 && down_stride % 8 == 0 && aligned16(wgu) && aligned16(wd);
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
     const dim3 grid_a(num_tokens * top, (ff + MOE_SPARSE_FEATURES - 1) / MOE_SPARSE_FEATURES);
     const dim3 grid_b(num_tokens, (W + MOE_SPARSE_FEATURES - 1) / MOE_SPARSE_FEATURES);
@@ -402,12 +425,12 @@ extern "C" int llm_moe_sparse(const void* x, int x_dtype, const void* wgu, const
         launch_pdl((moe_gate_up_sparse_kernel<float, float, float>), grid_a, block, smem_a, s, static_cast<const float*>(x),
                    static_cast<const float*>(wgu), ids, weights, static_cast<float*>(act), W, ff, top, limit, alpha, vec, shift);
         launch_pdl((moe_down_sparse_kernel<float, float>), grid_b, block, smem_b, s, static_cast<const float*>(act),
-                   static_cast<const float*>(wd), ids, out, W, ff, top, E, vec);
+                   static_cast<const float*>(wd), ids, out, W, ff, top, down_stride, vec);
     } else if (x_dtype == LLM_DT_BF16) {
         launch_pdl((moe_gate_up_sparse_kernel<bf16, bf16, bf16>), grid_a, block, smem_a, s, static_cast<const bf16*>(x),
                    static_cast<const bf16*>(wgu), ids, weights, static_cast<bf16*>(act), W, ff, top, limit, alpha, vec, shift);
         launch_pdl((moe_down_sparse_kernel<bf16, bf16>), grid_b, block, smem_b, s, static_cast<const bf16*>(act),
-                   static_cast<const bf16*>(wd), ids, out, W, ff, top, E, vec);
+                   static_cast<const bf16*>(wd), ids, out, W, ff, top, down_stride, vec);
     } else {
         return LLM_REFUSED_DTYPE;
     }
@@ -500,12 +523,13 @@ __global__ void moe_act_pairs_kernel(const T* __restrict__ gu, const int32_t* __
 
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ y, const int32_t* __restrict__ pos, float* __restrict__ out,
-                                   int W, int top, int vec) {
+                                   int W, int top, int vec, const float* __restrict__ base) {
     pdl_begin();
     const long long t = blockIdx.x;
     if (vec) {
         for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 8; i < W; i += gridDim.y * blockDim.x * 8) {
             float acc[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+            if (base) load8(base + t * W + i, acc);
             for (int k = 0; k < top; ++k) {
                 const int r = pos[t * top + k];
                 if (r < 0) continue;
@@ -518,7 +542,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const int32_t* __res
         }
     } else {
         for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
-            float acc = 0.0f;
+            float acc = base ? base[t * W + i] : 0.0f;
             for (int k = 0; k < top; ++k) {
                 const int r = pos[t * top + k];
                 if (r >= 0) acc += to_f32(y[static_cast<size_t>(r) * W + i]);
@@ -538,7 +562,8 @@ extern "C" int llm_moe_sort(const int32_t* ids, int pairs, int E, int32_t* offs,
 }
 
 // which = 0: gather (a = x [T, W], out = xs [pairs, W]); 1: activation (a = gu [pairs, 2 n], out = act [pairs, n]);
-// 2: combine (a = y [pairs, n], out = float32 [T, n], index = pos).  n is the row width of `out`.
+// 2: combine (a = y [pairs, n], out = float32 [T, n], index = pos, `weights` an optional float32
+// [T, n] the sums start from, aligned like `out`).  n is the row width of `out`.
 extern "C" int llm_moe_rows(int which, const void* a, int dtype, const int32_t* index, const float* weights, void* out,
                             int rows, int n, int top, float limit, float alpha, float shift, uintptr_t stream) {
     if (rows <= 0) return LLM_OK;
@@ -562,9 +587,9 @@ extern "C" int llm_moe_rows(int which, const void* a, int dtype, const int32_t* 
         else return LLM_REFUSED_DTYPE;
     } else {
         if (dtype == LLM_DT_F32) launch_pdl((moe_combine_kernel<float>), grid, block, 0, s, static_cast<const float*>(a), index,
-                                            static_cast<float*>(out), n, top, vec);
+                                            static_cast<float*>(out), n, top, vec, weights);
         else if (dtype == LLM_DT_BF16) launch_pdl((moe_combine_kernel<bf16>), grid, block, 0, s, static_cast<const bf16*>(a), index,
-                                                  static_cast<float*>(out), n, top, vec);
+                                                  static_cast<float*>(out), n, top, vec, weights);
         else return LLM_REFUSED_DTYPE;
     }
     return launch_status();

@@ -181,6 +181,28 @@ def embedding_sinusoid(ids: torch.Tensor, table: torch.Tensor, positions: torch.
     return out, copy
 
 
+def embedding_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                   center: bool, status: torch.Tensor, feedback: Optional[torch.Tensor] = None,
+                   copy_dtype: Optional[torch.dtype] = None):
+    """float32 [T, H] = norm(table[ids]) * weight (+ bias), layer norm (`center`) or RMS norm.  With `copy_dtype` the same
+    rows come back a second time in that dtype.  Returns (stream, copy or None)."""
+    _dev(ids, table, weight, bias, status, feedback)
+    _i32(ids, "ids")
+    T, (V, H) = ids.numel(), table.shape
+    for t in (weight, bias):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != H):
+            raise KernelError("the norm's weight and bias must be float32 of the row length")
+    out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    copy = torch.empty((T, H), dtype=copy_dtype, device=table.device) if copy_dtype is not None else None
+    f = _fn("embedding", "llm_embedding_norm",
+            [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+             c_void_p, c_int, c_void_p])
+    _check(f(_ptr(ids), _ptr(table), _dt(table), _ptr(weight), _ptr(bias), float(eps), 1 if center else 0, _ptr(out), _ptr(copy),
+             _dt(copy) if copy is not None else 0, T, H, V, _ptr(status), _ptr(feedback),
+             feedback.numel() if feedback is not None else 0, _stream()), "embedding_norm")
+    return out, copy
+
+
 def scatter_int32(dst: torch.Tensor, index: torch.Tensor, value: torch.Tensor, count: torch.Tensor,
                   max_count: int, status: torch.Tensor) -> None:
     """dst.flat[index[i]] = value[i] for i < count[0] (count is a device scalar; None: for i < max_count)."""
@@ -537,6 +559,18 @@ def gate_mul(a: torch.Tensor, gate: Optional[torch.Tensor], gate_off: int, out: 
              out_off, T, w, {None: 0, "sigmoid": 1, "silu": 2}[kind], float(scale), int(per_head), _stream()), "gate_mul")
 
 
+def _sinks(sink, nq: int, device) -> Optional[torch.Tensor]:
+    """A softmax sink as the kernels take it: float32 [heads].  A number stands for all heads."""
+    if sink is None:
+        return None
+    if not isinstance(sink, torch.Tensor):
+        return torch.full((nq,), float(sink), dtype=torch.float32, device=device)
+    _dev(sink)
+    if sink.dtype != torch.float32 or sink.numel() != nq:
+        raise KernelError("sinks must be float32 [heads]")
+    return sink
+
+
 def paged_attention_generic_kv(q: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, positions, token_entry,
                                entry_slot, block_table: torch.Tensor, nq: int, nkv: int, dk: int, dv: int,
                                page_size: int, window: Optional[int], scale: float, status: torch.Tensor,
@@ -545,7 +579,7 @@ def paged_attention_generic_kv(q: torch.Tensor, keys: torch.Tensor, values: torc
                                gate_per_head: bool = False, rows: Optional[torch.Tensor] = None,
                                head_scale: Optional[torch.Tensor] = None, log_bias=None,
                                values_in_keys: bool = False, keep_first: int = 0,
-                               sink: Optional[float] = None) -> torch.Tensor:
+                               sink=None) -> torch.Tensor:
     """Causal attention of every token in q [T, nq*dk] over its request's pages of `keys` [pages, nkv, page,
     dk] and `values` [pages, nkv, page, dv] (views with any page stride), written into columns out_off ..
     out_off + nq*dv of `out`, times sigmoid(gate[:, gate_off + ...]) (float32, optional; one value per output
@@ -554,8 +588,8 @@ def paged_attention_generic_kv(q: torch.Tensor, keys: torch.Tensor, values: torc
     (-1 entries are padding).  `head_scale` (float32 [nq]) multiplies each head's scaled scores; `log_bias` = (r1, r2),
     float32 [nq] each, takes r1[h] * ln(1 + r2[h] * (i - j)) off them.  `values_in_keys`: `values` is None and the
     values are the first dv entries of the key rows.  `keep_first`: with a window, the sequence's first so many keys
-    stay visible to every later query.  `sink`: a score whose exponential joins the softmax's denominator without a
-    value (None: ordinary softmax)."""
+    stay visible to every later query.  `sink`: a score (one number, or float32 [nq]: one per head) whose exponential joins
+    the softmax's denominator without a value (None: ordinary softmax)."""
     r1, r2 = log_bias if log_bias is not None else (None, None)
     _dev(q, positions, token_entry, entry_slot, block_table, status, dist_bias, rows, head_scale, r1, r2)
     _i32(rows, "rows")
@@ -582,7 +616,8 @@ def paged_attention_generic_kv(q: torch.Tensor, keys: torch.Tensor, values: torc
             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p,
              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_longlong,
              c_int, c_float, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_longlong, c_int, c_int, c_float, c_void_p])
+             c_longlong, c_int, c_void_p, c_void_p])
+    sinks = _sinks(sink, nq, q.device)
     _check(f(_ptr(q), _ptr(out), _dt(q), _ptr(keys), _ptr(values), _dt(keys), keys.stride(0), values.stride(0),
              _ptr(positions), _ptr(token_entry), _ptr(entry_slot), _ptr(block_table), block_table.shape[1],
              rows.numel() if rows is not None else T, nq, nkv,
@@ -590,7 +625,7 @@ def paged_attention_generic_kv(q: torch.Tensor, keys: torch.Tensor, values: torc
              gate.stride(0) if gate is not None else 0, gate_off, float(out_scale), out.stride(0), out_off,
              _ptr(status), _ptr(dist_bias), dist_bias.shape[0] if dist_bias is not None else 0,
              1 if gate_per_head else 0, _ptr(rows), _ptr(head_scale), _ptr(r1), _ptr(r2), value_row,
-             int(keep_first) if window else 0, 0 if sink is None else 1, float(sink or 0.0), _stream()),
+             int(keep_first) if window else 0, _ptr(sinks), _stream()),
            "paged_attention_generic_kv")
     return out
 
@@ -944,21 +979,91 @@ def recur_chain(state: torch.Tensor, head_stride: int, scratch_s: torch.Tensor, 
              1 if normaliser else 0, head_stride, state.stride(0), _stream()), "recur_chain")
 
 
+# ---- the gated delta rule ---------------------------------------------------------------------------------
+def delta_padded(d: int) -> int:
+    """Rows a head's state is padded to in the delta rule's kernels (0: they do not take this key width)."""
+    return int(_fn("delta_rule", "llm_delta_padded", [c_int])(d))
+
+
+def delta_supported(d: int, v: int) -> bool:
+    return bool(_fn("delta_rule", "llm_delta_supported", [c_int, c_int])(d, v))
+
+
+def delta_rule(proj: torch.Tensor, offs, ranks, conv_w: torch.Tensor, w_decay: torch.Tensor, w_gate: torch.Tensor,
+               dt_bias: torch.Tensor, a_log: torch.Tensor, norm_w: torch.Tensor, eps: float, out_scale: float, out: torch.Tensor,
+               out_off: int, state: torch.Tensor, batch, H: int, G: int, D: int, V: int, single: bool = False) -> None:
+    """The gated delta rule over a step's tokens, from the float32 projection to the gated, normed heads in columns
+    out_off .. out_off + H * V of `out` (see csrc/delta_rule.cu for the arithmetic and the layout of `state` [slots, n]).
+    `offs` = columns of (q | k | v side by side, step sizes, first half of the decays, first half of the gates), `ranks` =
+    (decay, gate); `conv_w` float32 [C, taps]; `w_decay` [rank, H * D] and `w_gate` [rank, H * V]: the second halves
+    transposed, both float32 or both bfloat16.  `single`: every entry brings one token (one kernel)."""
+    _dev(conv_w, w_decay, w_gate, dt_bias, a_log, norm_w, state, batch.positions, batch.token_entry, batch.entry_slot,
+         batch.entry_q_start, batch.entry_q_len)
+    q_off, b_off, a_off, g_off = offs
+    ra, rg = ranks
+    C, taps = conv_w.shape
+    if (proj.dtype != torch.float32 or proj.stride(1) != 1 or state.dtype != torch.float32 or out.stride(1) != 1
+            or any(t.dtype != torch.float32 for t in (conv_w, dt_bias, a_log, norm_w))):
+        raise KernelError("delta_rule: float32 projection, state, convolutions, biases and norm weight")
+    if (C != 2 * G * D + H * V or tuple(w_decay.shape) != (ra, H * D) or tuple(w_gate.shape) != (rg, H * V)
+            or w_decay.dtype != w_gate.dtype or dt_bias.numel() != H * D or a_log.numel() != H or norm_w.numel() != V):
+        raise KernelError("delta_rule: a weight of the wrong size")
+    if max(q_off + C, b_off + H, a_off + ra, g_off + rg) > proj.shape[1] or out_off + H * V > out.shape[1]:
+        raise KernelError("delta_rule: the projection or the output is narrower than its pieces")
+    T, dev = proj.shape[0], proj.device
+    head = [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p,
+            c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_longlong, c_int, c_void_p, c_longlong, c_void_p]
+    args = (_ptr(proj), proj.stride(0), q_off, b_off, a_off, ra, g_off, rg, _ptr(conv_w), taps, _ptr(w_decay), _ptr(w_gate),
+            _dt(w_decay), _ptr(dt_bias), _ptr(a_log), _ptr(norm_w), float(eps), float(out_scale), _ptr(out), _dt(out),
+            out.stride(0), out_off, _ptr(state), state.stride(0), _ptr(batch.positions))
+    if single:
+        f = _fn("delta_rule", "llm_delta_step", head + [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+        _check(f(*args, _ptr(batch.entry_slot), _ptr(batch.entry_q_start), batch.num_entries, H, G, D, V, _stream()), "delta_step")
+        return
+    DP, VP = delta_padded(D), (V + 3) // 4 * 4
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
+    qn, kn, vn, kq, beta = new(T, G, DP), new(T, G, DP), new(T, H, VP), new(T, G), new(T, H)
+    decay = new(T, H, DP) if D == DP else torch.zeros((T, H, DP), dtype=torch.float32, device=dev)
+    gate, o = new(T, H, V), new(T, H, V)
+    f = _fn("delta_rule", "llm_delta_scan",
+            head + [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int] + [c_void_p] * 9)
+    _check(f(*args, _ptr(batch.token_entry), _ptr(batch.entry_slot), _ptr(batch.entry_q_start), _ptr(batch.entry_q_len), T,
+             batch.num_entries, H, G, D, V, _ptr(qn), _ptr(kn), _ptr(vn), _ptr(kq), _ptr(beta), _ptr(decay), _ptr(gate), _ptr(o),
+             _stream()), "delta_scan")
+    global launch_count
+    launch_count += 3                          # four kernels in one call
+
+
 # ---- several residual streams ----------------------------------------------------------------------------
 def stream_norm(streams: torch.Tensor, y, mix: Optional[torch.Tensor], outw: Optional[torch.Tensor],
                 inw: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, center: bool,
                 out_dtype: Optional[torch.dtype], rows: Optional[torch.Tensor] = None,
-                write_back: bool = True, fan: bool = False) -> Optional[torch.Tensor]:
+                write_back: bool = True, fan: bool = False, bias: Optional[torch.Tensor] = None, y2=None,
+                source: Optional[torch.Tensor] = None, add: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """streams: float32 [S, T, H] (or [T, H]: one stream).  With y (a sublayer's output that has not been added
     yet, possibly an `ops.PartialSum`): x_t <- sum_s mix[s, t] x_s + outw[t] * y for all t (mix None: the identity,
     outw None: ones), written back unless `rows` is given.  Then, with `weight`: the norm (`center`: layer norm,
     else RMS norm) of u = sum_t inw[t] x_t (inw None: the plain sum) times `weight`, returned in `out_dtype` for
     all rows or for `rows`.  `fan`: only streams[0] holds data yet (a model's embedding); every stream is read from
-    there and written to its own place."""
+    there and written to its own place.  `bias` (float32 [H]) is added after the weight.  `y2`: a second output that
+    joins as y does.  One stream only: `source` (float32 [T, H]) is read in the stream's place and `add` (float32 [H])
+    joins every row (source + add + y is then the new stream).  Without `weight` but with `out_dtype`: the sum of the
+    streams itself, unnormalised."""
     parts, part_stride = 1, 0
     if isinstance(y, PartialSum):
         parts, part_stride = y.parts.shape[0], y.parts.stride(0)
         y = y.parts[0]
+    parts2, part_stride2 = 1, 0
+    if isinstance(y2, PartialSum):
+        parts2, part_stride2 = y2.parts.shape[0], y2.parts.stride(0)
+        y2 = y2.parts[0]
+    _dev(bias, y2, source, add)
+    if y2 is not None and (y is None or y2.dtype != y.dtype or y2.shape != y.shape):
+        raise KernelError("a second output must look like the first")
+    if (source is not None or add is not None) and (y is None or streams.dim() != 2):
+        raise KernelError("a source or an added row needs one stream and an output that joins it")
+    if source is not None and (source.dtype != torch.float32 or source.shape != streams.shape):
+        raise KernelError("the source must look like the stream")
     if fan and (y is not None or rows is not None):
         raise KernelError("stream_norm: the first fan-out takes no pending update and no row selection")
     _dev(streams, y, mix, outw, inw, weight, rows)
@@ -967,54 +1072,63 @@ def stream_norm(streams: torch.Tensor, y, mix: Optional[torch.Tensor], outw: Opt
         raise KernelError("the residual streams are float32")
     S = streams.shape[0] if streams.dim() == 3 else 1
     T, H = streams.shape[-2], streams.shape[-1]
-    for t, n in ((mix, S * S), (outw, S), (inw, S), (weight, H)):
+    for t, n in ((mix, S * S), (outw, S), (inw, S), (weight, H), (bias, H), (add, H)):
         if t is not None and (t.dtype != torch.float32 or t.numel() != n):
             raise KernelError("stream_norm: a coefficient tensor of the wrong size or type")
     if y is not None and tuple(y.shape) != (T, H):
         raise KernelError("y must have a stream's shape")
     n = rows.numel() if rows is not None else T
-    out = torch.empty((n, H), dtype=out_dtype, device=streams.device) if weight is not None else None
+    out = torch.empty((n, H), dtype=out_dtype, device=streams.device) if out_dtype is not None else None
     f = _fn("streams", "llm_stream_norm",
             [c_void_p, c_longlong, c_longlong, c_int, c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_float, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+             c_float, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p,
+             c_void_p])
     _check(f(_ptr(streams), T * H, 0 if fan else T * H, S, _ptr(y), _dt(y) if y is not None else 0, parts, part_stride, _ptr(mix), _ptr(outw),
              _ptr(inw), _ptr(weight), float(eps), 1 if center else 0, _ptr(out), _dt(out) if out is not None else 0,
-             _ptr(rows), n, H, 1 if (write_back and rows is None and (y is not None or fan)) else 0, _stream()), "stream_norm")
+             _ptr(rows), n, H, 1 if (write_back and rows is None and (y is not None or fan)) else 0, _ptr(bias), _ptr(y2), parts2,
+             part_stride2, _ptr(source), _ptr(add), _stream()), "stream_norm")
     return out
 
 
 # ---- routed experts ----------------------------------------------------------------------------------------
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, groups, route_scale: float, lists: bool = False,
-              score: str = "sigmoid", correction: Optional[torch.Tensor] = None, identity: int = 0):
+              score: str = "sigmoid", correction: Optional[torch.Tensor] = None, identity: int = 0,
+              bias: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None):
     """Per token of x [T, W]: scores of `w_router` (float32 [E, W]; `score` 'sigmoid', or 'softmax' over all E), the
     `top` best among the experts of the best groups (`groups` = (count, keep) or None), weights normalised and
     scaled.  `correction` (float32 [E]) is added to the scores for the choice only.  The last `identity` router
     outputs are no experts: a token that picks one gets its own input back times the weight.  Returns the dense
     float32 weights [T, E - identity] (zero where not chosen) and, with `lists`, ids int32 [T, top] (-1 for an
-    identity pick) and weights float32 [T, top]; with `identity`, also the float32 [T] share of a token's own input."""
-    _dev(x, w_router, correction)
+    identity pick) and weights float32 [T, top]; with `identity`, also the float32 [T] share of a token's own input.
+    `bias` (float32 [E]) joins the logits before the score.  `shared_gate` (float32 [W]): the sigmoid of its product with
+    the token comes back too, as the last member, float32 [T] (the weight of an expert that every token runs)."""
+    _dev(x, w_router, correction, bias, shared_gate)
     T, W = x.shape
     E = w_router.shape[0]
     if w_router.dtype != torch.float32 or w_router.shape[1] != W:
         raise KernelError("the router's matrix must be float32 [experts, hidden]")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
         raise KernelError("the router's correction must be float32 [router outputs]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != E):
+        raise KernelError("the router's bias must be float32 [router outputs]")
+    if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.numel() != W):
+        raise KernelError("the shared expert's gate must be float32 [hidden]")
     if score not in ("sigmoid", "softmax") or not 0 <= identity < E:
         raise KernelError("score 'sigmoid' or 'softmax'; identity outputs fewer than the router's")
     dense = torch.empty((T, E - identity), dtype=torch.float32, device=x.device)
     idw = torch.empty((T,), dtype=torch.float32, device=x.device) if identity else None
+    share = torch.empty((T,), dtype=torch.float32, device=x.device) if shared_gate is not None else None
     ids = torch.empty((T, top), dtype=torch.int32, device=x.device) if lists else None
     wts = torch.empty((T, top), dtype=torch.float32, device=x.device) if lists else None
     count, keep = groups if groups is not None else (0, 0)
     f = _fn("moe", "llm_moe_route",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-             c_int, c_void_p, c_int, c_void_p, c_void_p])
+             c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
     _check(f(_ptr(x), _dt(x), _ptr(w_router), _ptr(dense), _ptr(ids), _ptr(wts), T, W, E, top, count, keep,
-             float(route_scale), 1 if score == "softmax" else 0, _ptr(correction), identity, _ptr(idw), _stream()), "moe_route")
-    out = (dense, ids, wts) if lists else dense
-    if identity:
-        return (out + (idw,)) if lists else (out, idw)
-    return out
+             float(route_scale), 1 if score == "softmax" else 0, _ptr(correction), identity, _ptr(idw), _ptr(bias),
+             _ptr(shared_gate), _ptr(share), _stream()), "moe_route")
+    out = ((dense, ids, wts) if lists else (dense,)) + ((idw,) if identity else ()) + ((share,) if share is not None else ())
+    return out if len(out) > 1 else dense
 
 
 def moe_finish(out: torch.Tensor, x: Optional[torch.Tensor], idw: Optional[torch.Tensor], shared=None) -> torch.Tensor:
@@ -1038,23 +1152,29 @@ def moe_finish(out: torch.Tensor, x: Optional[torch.Tensor], idw: Optional[torch
     return out
 
 
-def moe_act(gate_up, dense: torch.Tensor, E: int, ff: int, limit: float, alpha: float,
-            out_dtype: torch.dtype, shift: float = 1.0) -> torch.Tensor:
-    """act [T, E*ff] = dense[t, e] * g * sigmoid(alpha g) * (u + shift), g = min(gate, limit), u = clamp(up, +-limit),
+def moe_act(gate_up, dense: Optional[torch.Tensor], E: int, ff: int, limit: float, alpha: float,
+            out_dtype: torch.dtype, shift: float = 1.0, shared=None) -> torch.Tensor:
+    """`shared` = (ff_s, limit_s, share): the rows of the product go on with a shared expert's 2 * ff_s columns, and those of
+    the result with its ff_s activations, times share[t] (float32 [T], None: one); E may then be 0.
+    act [T, E*ff] = dense[t, e] * g * sigmoid(alpha g) * (u + shift), g = min(gate, limit), u = clamp(up, +-limit),
     from the float32 product [T, E*2*ff] (per expert: ff gate columns, then ff up columns; may be a `PartialSum`)."""
     parts, part_stride = 1, 0
     if isinstance(gate_up, PartialSum):
         parts, part_stride = gate_up.parts.shape[0], gate_up.parts.stride(0)
         gate_up = gate_up.parts[0]
-    _dev(gate_up, dense)
+    ffs, limit_s, share = shared if shared is not None else (0, 1.0, None)
+    _dev(gate_up, dense, share)
     T = gate_up.shape[0]
-    if gate_up.dtype != torch.float32 or gate_up.shape[1] != 2 * E * ff or tuple(dense.shape) != (T, E):
-        raise KernelError("moe_act wants the float32 product [T, experts * 2 * ff] and the weights [T, experts]")
-    act = torch.empty((T, E * ff), dtype=out_dtype, device=gate_up.device)
+    if gate_up.dtype != torch.float32 or gate_up.shape[1] != 2 * (E * ff + ffs) or (E > 0 and tuple(dense.shape) != (T, E)):
+        raise KernelError("moe_act wants the float32 product [T, experts * 2 * ff (+ 2 * ff_s)] and the weights [T, experts]")
+    if share is not None and (share.dtype != torch.float32 or share.numel() != T):
+        raise KernelError("the shared expert's weights must be float32 [T]")
+    act = torch.empty((T, E * ff + ffs), dtype=out_dtype, device=gate_up.device)
     f = _fn("moe", "llm_moe_act",
-            [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p])
+            [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_float,
+             c_void_p, c_void_p])
     _check(f(_ptr(gate_up), parts, part_stride, _ptr(dense), _ptr(act), _dt(act), T, E, ff, float(limit), float(alpha),
-             float(shift), _stream()), "moe_act")
+             float(shift), ffs, float(limit_s), _ptr(share), _stream()), "moe_act")
     return act
 
 
@@ -1063,21 +1183,21 @@ def moe_sparse(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, i
     """The routed feed-forward for steps of few tokens: only the chosen experts' matrices are read.  x [T, W] and
     the matrices in one dtype (bfloat16 or float32); `ids`, `weights` [T, top] from `moe_route`.  Returns the
     float32 sum [T, W] of the chosen experts' weighted outputs."""
-    _dev(x, w_gate_up, w_down, ids, weights)
+    _dev(x, w_gate_up, ids, weights)
     _i32(ids, "ids")
     T, W = x.shape
     top = ids.shape[1]
     E = w_gate_up.shape[0] // (2 * ff)
-    if (w_gate_up.shape != (E * 2 * ff, W) or w_down.shape != (W, E * ff) or w_gate_up.dtype != x.dtype
+    if (w_gate_up.shape != (E * 2 * ff, W) or w_down.shape != (W, E * ff) or not w_down.is_cuda or w_down.stride(1) != 1 or w_gate_up.dtype != x.dtype
             or w_down.dtype != x.dtype or weights.dtype != torch.float32):
         raise KernelError("moe_sparse: x, [E*2*ff, W] and [W, E*ff] in one dtype, float32 weights [T, top]")
     act = torch.empty((T * top, ff), dtype=x.dtype, device=x.device)
     out = torch.empty((T, W), dtype=torch.float32, device=x.device)
     f = _fn("moe", "llm_moe_sparse",
             [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-             c_int, c_float, c_float, c_float, c_void_p])
+             c_int, c_float, c_float, c_float, c_longlong, c_void_p])
     code = f(_ptr(x), _dt(x), _ptr(w_gate_up), _ptr(w_down), _dt(w_down), _ptr(ids), _ptr(weights), _ptr(act), _ptr(out),
-             T, W, ff, E, top, float(limit), float(alpha), float(shift), _stream())
+             T, W, ff, E, top, float(limit), float(alpha), float(shift), w_down.stride(0), _stream())
     _check(code, "moe_sparse")
     global launch_count
     launch_count += 1                      # two kernels in one call
@@ -1090,14 +1210,16 @@ def grouped_product_available() -> bool:
 
 
 def moe_sorted(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-               E: int, ff: int, limit: float, alpha: float, shift: float = 1.0) -> torch.Tensor:
-    """The routed feed-forward for prompt portions: the (token, choice) pairs are sorted by expert (the engine's
+               E: int, ff: int, limit: float, alpha: float, shift: float = 1.0, base: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """`base` (float32 [T, W]): the sums start from it.  The routed feed-forward for prompt portions: the (token, choice) pairs are sorted by expert (the engine's
     kernels), each expert's rows go through ITS matrices in the library's grouped matrix product (bfloat16 in,
     bfloat16 out, 32-bit accumulation; the row offsets stay on the device), the activation takes each row's
     routing weight, and a token's rows are added in 32-bit.  Returns float32 [T, W]."""
-    _dev(x, w_gate_up, w_down, ids, weights)
+    _dev(x, w_gate_up, ids, weights, base)
     T, W = x.shape
     top = ids.shape[1]
+    if base is not None and (base.dtype != torch.float32 or tuple(base.shape) != (T, W)):
+        raise KernelError("moe_sorted: the base must be float32 [T, W]")
     pairs = T * top
     dev = x.device
     offs = torch.empty(E, dtype=torch.int32, device=dev)
@@ -1113,9 +1235,9 @@ def moe_sorted(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, i
     act = torch.empty((pairs, ff), dtype=x.dtype, device=dev)
     _check(rows_fn(1, _ptr(gu), _dt(gu), _ptr(row_pair), _ptr(weights), _ptr(act), pairs, ff, top, float(limit), float(alpha),
                    float(shift), _stream()), "moe_act_pairs")
-    y = torch._grouped_mm(act, w_down.view(W, E, ff).permute(1, 2, 0), offs=offs)
+    y = torch._grouped_mm(act, w_down.as_strided((E, ff, W), (ff, 1, w_down.stride(0)), w_down.storage_offset()), offs=offs)
     out = torch.empty((T, W), dtype=torch.float32, device=dev)
-    _check(rows_fn(2, _ptr(y), _dt(y), _ptr(pos), None, _ptr(out), T, W, top, 0.0, 0.0, 0.0, _stream()), "moe_combine")
+    _check(rows_fn(2, _ptr(y), _dt(y), _ptr(pos), _ptr(base), _ptr(out), T, W, top, 0.0, 0.0, 0.0, _stream()), "moe_combine")
     return out
 
 
@@ -1152,7 +1274,7 @@ def paged_attention_decode(q: torch.Tensor, out: torch.Tensor, cache: torch.Tens
                            n_rows: int, positions, token_entry, entry_slot, block_table: torch.Tensor, nq: int,
                            nkv: int, d: int, page_size: int, window: Optional[int], scale: float, num_splits: int,
                            status: torch.Tensor, dist_bias_t: Optional[torch.Tensor] = None,
-                           analytic_bias: bool = False, keep_first: int = 0, sink: Optional[float] = None) -> torch.Tensor:
+                           analytic_bias: bool = False, keep_first: int = 0, sink=None) -> torch.Tensor:
     """Attention for single decoded tokens (rows of q named by `rows`, or rows 0..n_rows-1), written
     into the same rows of `out`.  bfloat16 only.  `dist_bias_t` float32 [nq, distances]: a bias by distance TIMES
     log2(e); row min(p - j, distances - 1) of a head joins the scaled score of the query at p and key j.
@@ -1176,12 +1298,13 @@ def paged_attention_decode(q: torch.Tensor, out: torch.Tensor, cache: torch.Tens
     scratch = decode_scratch(q.device, int(need))
     f = _fn("attention_decode", "llm_paged_attention_decode_ex",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-             c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
+             c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
              c_void_p])
+    sinks = _sinks(sink, nq, q.device)
     _check(f(_ptr(q), _ptr(out), _ptr(cache), _ptr(rows), n_rows, _ptr(positions), _ptr(token_entry),
              _ptr(entry_slot), _ptr(block_table), block_table.shape[1], nq, nkv, d, page_size,
              int(window) if window else 0, float(scale), cache.shape[0], num_splits, _ptr(scratch), _ptr(status),
-             _ptr(dist_bias_t), dist_len, keep_first, 0 if sink is None else 1, float(sink or 0.0), _stream()),
+             _ptr(dist_bias_t), dist_len, keep_first, _ptr(sinks), _stream()),
            "paged_attention_decode")
     if num_splits > 1:
         global launch_count
@@ -1223,7 +1346,7 @@ def paged_attention_prefill_biased(q: torch.Tensor, out: torch.Tensor, out_off: 
                                    window: Optional[int], scale: float, status: torch.Tensor,
                                    dist_bias_t: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None,
                                    gate_off: int = 0, out_scale: float = 1.0, analytic_bias: bool = False,
-                                   keep_first: int = 0, sink: Optional[float] = None) -> torch.Tensor:
+                                   keep_first: int = 0, sink=None) -> torch.Tensor:
     """`keep_first`: with a window, the sequence's first so many keys stay visible to every later query.  `sink`: a score
     whose exponential joins the softmax's denominator without a value.  `analytic_bias`: `dist_bias_t` is float32 [nq, 3], per head a temperature on the scaled score and the numbers
     r1, r2 of the bias r1 * ln(1 + r2 * (i - j)) that is taken off it (evaluated in the kernel; no table).
@@ -1246,13 +1369,14 @@ def paged_attention_prefill_biased(q: torch.Tensor, out: torch.Tensor, out_off: 
     f = _fn("attention_prefill", "llm_paged_attention_prefill_ex",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
              c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int,
-             c_float, c_longlong, c_int, c_int, c_int, c_float, c_void_p])
+             c_float, c_longlong, c_int, c_int, c_void_p, c_void_p])
+    sinks = _sinks(sink, nq, q.device)
     _check(f(_ptr(q), _ptr(out), _ptr(cache), _ptr(tiles), n_tiles, _ptr(entry_slot), _ptr(entry_q_start),
              _ptr(entry_q_len), _ptr(entry_kv_len), _ptr(block_table), block_table.shape[1], nq, nkv, d,
              page_size, int(window) if window else 0, float(scale), cache.shape[0], _ptr(status), _ptr(dist_bias_t),
              dist_len, _ptr(head_gate),
              head_gate.stride(0) if head_gate is not None else 0, gate_off, float(out_scale), out.stride(0), out_off,
-             int(keep_first) if window else 0, 0 if sink is None else 1, float(sink or 0.0),
+             int(keep_first) if window else 0, _ptr(sinks),
              _stream()), "paged_attention_prefill_biased")
     return out
 

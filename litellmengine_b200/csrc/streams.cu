@@ -12,7 +12,11 @@
 // `mix` is the identity, a null `outw` or `inw` all ones (in = ones: the sum of the streams, which is what
 // the model's final norm reads).  `rows` picks the rows that are read (the final norm runs only where
 // logits are wanted); the new streams are written back only without `rows`.  A null `w`: the streams are
-// updated and nothing is normalised.  `read_stride` is the distance between the streams as they are READ: 0 at a
+// updated and nothing is normalised; u itself is written when there is an `out` (a copy of the new stream in the
+// compute dtype).  `b`: a bias added after the weight.  `y2` (the type of y, k-splits of its own): a second sublayer
+// output that joins by the same coefficients as y (a layer whose sublayers run side by side).  `source` (S = 1): the
+// stream is read from there instead of from `streams`, and `add` [hidden] is added to every row on the way (the start
+// of a pass of a looped span: source + add + y become the new stream).  `read_stride` is the distance between the streams as they are READ: 0 at a
 // model's first layer, where all streams equal the embedding that sits in stream 0 (they are then written out
 // to their own places, so no kernel has to copy the embedding S times).
 //
@@ -57,7 +61,9 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
                                    const TY* __restrict__ y, int y_parts, long long y_part_stride,
                                    const float* __restrict__ mix, const float* __restrict__ outw,
                                    const float* __restrict__ inw, const float* __restrict__ w, float eps, int center,
-                                   TO* __restrict__ out, const int32_t* __restrict__ rows, int hidden, int write_back, int vec) {
+                                   TO* __restrict__ out, const int32_t* __restrict__ rows, int hidden, int write_back, int vec,
+                                   const float* __restrict__ b, const TY* __restrict__ y2, int y2_parts, long long y2_part_stride,
+                                   const float* __restrict__ source, const float* __restrict__ add) {
     extern __shared__ __align__(16) float smem[];
     float* u = smem;                                   // [hidden]
     float* scratch = smem + ((hidden + 7) & ~7);       // 33
@@ -72,7 +78,9 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
     __syncthreads();
     const size_t src = rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
     float* xr = streams + src * hidden;
+    const float* xs = source ? source + src * hidden : xr;
     const TY* yr = y ? y + src * hidden : nullptr;
+    const TY* y2r = y2 ? y2 + src * hidden : nullptr;
     TO* orow = out ? out + static_cast<size_t>(blockIdx.x) * hidden : nullptr;
     float sum = 0.0f;
     // four neighbouring columns a thread and trip when the rows allow sixteen-byte accesses, else one
@@ -83,12 +91,19 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
         for (int s = 0; s < SM; ++s)
             if (s < S) {
                 if (vec) {
-                    const float4 v = *reinterpret_cast<const float4*>(xr + s * read_stride + h);
+                    const float4 v = *reinterpret_cast<const float4*>(xs + s * read_stride + h);
                     x[s][0] = v.x; x[s][1] = v.y; x[s][2] = v.z; x[s][3] = v.w;
                 } else {
-                    x[s][0] = xr[s * read_stride + h];
+                    x[s][0] = xs[s * read_stride + h];
                 }
             }
+        if (SM == 1 && add) {
+            float one[4];
+            stream_load4(add + h, one, vec);
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+                if (c == 0 || vec) x[0][c] += one[c];
+        }
         float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         if (yr) {
             float yv[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -98,6 +113,13 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
 #pragma unroll
                 for (int c = 0; c < 4; ++c) yv[c] += one[c];
             }
+            if (y2r)
+                for (int part = 0; part < y2_parts; ++part) {
+                    float one[4];
+                    stream_load4(y2r + part * y2_part_stride + h, one, vec);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) yv[c] += one[c];
+                }
 #pragma unroll
             for (int t = 0; t < SM; ++t)
                 if (t < S) {
@@ -130,7 +152,12 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
                     }
                 }
         }
-        if (vec) {
+        if (!w) {                                       // no norm: the stream itself, if anybody wants it
+            if (orow) {
+                if (vec) stream_store4(orow + h, acc[0], acc[1], acc[2], acc[3]);
+                else orow[h] = from_f32<TO>(acc[0]);
+            }
+        } else if (vec) {
             *reinterpret_cast<float4*>(u + h) = make_float4(acc[0], acc[1], acc[2], acc[3]);
             sum += (acc[0] + acc[1]) + (acc[2] + acc[3]);
         } else {
@@ -157,10 +184,11 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
         if (vec) {
             const float4 g = *reinterpret_cast<const float4*>(w + h);
             const float4 a = *reinterpret_cast<const float4*>(u + h);
-            stream_store4(orow + h, (a.x - mean) * inv * g.x, (a.y - mean) * inv * g.y, (a.z - mean) * inv * g.z,
-                          (a.w - mean) * inv * g.w);
+            const float4 e = b ? *reinterpret_cast<const float4*>(b + h) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            stream_store4(orow + h, (a.x - mean) * inv * g.x + e.x, (a.y - mean) * inv * g.y + e.y,
+                          (a.z - mean) * inv * g.z + e.z, (a.w - mean) * inv * g.w + e.w);
         } else {
-            orow[h] = from_f32<TO>((u[h] - mean) * inv * w[h]);
+            orow[h] = from_f32<TO>((u[h] - mean) * inv * w[h] + (b ? b[h] : 0.0f));
         }
     }
 }
@@ -168,11 +196,15 @@ __global__ void stream_norm_kernel(float* __restrict__ streams, long long stream
 extern "C" int llm_stream_norm(float* streams, long long stream_stride, long long read_stride, int S, const void* y, int y_dtype, int y_parts,
                                long long y_part_stride, const float* mix, const float* outw, const float* inw,
                                const float* w, float eps, int center, void* out, int out_dtype, const int32_t* rows,
-                               int num_rows, int hidden, int write_back, uintptr_t stream) {
+                               int num_rows, int hidden, int write_back, const float* b, const void* y2, int y2_parts,
+                               long long y2_part_stride, const float* source, const float* add, uintptr_t stream) {
     if (num_rows <= 0) return LLM_OK;
     if (hidden <= 0 || S < 1 || S > ST_MAX) return LLM_REFUSED_SIZE;
     if (write_back && rows) return LLM_REFUSED_SIZE;
     if (w && !out) return LLM_REFUSED_SIZE;
+    if ((source || add) && (S != 1 || !y)) return LLM_REFUSED_SIZE;
+    if (y2 && !y) return LLM_REFUSED_SIZE;
+    if (y2_parts < 1) y2_parts = 1;
     const size_t smem = (static_cast<size_t>((hidden + 7) & ~7) + 33 + S * S + 2 * S) * sizeof(float);
     if (smem > 200 * 1024) return LLM_REFUSED_SIZE;
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
@@ -182,7 +214,9 @@ extern "C" int llm_stream_norm(float* streams, long long stream_stride, long lon
     if (num_rows <= 256 && hidden > 4 * threads) threads = hidden / 4 >= 512 ? 512 : ((hidden / 4 + 31) / 32) * 32;
     if (y_parts < 1) y_parts = 1;
     const int vec = hidden % 4 == 0 && aligned16(streams) && stream_stride % 4 == 0 && read_stride % 4 == 0 &&
-                    (!y || (aligned16(y) && y_part_stride % 4 == 0)) && (!w || aligned16(w)) && (!out || aligned16(out));
+                    (!y || (aligned16(y) && y_part_stride % 4 == 0)) && (!w || aligned16(w)) && (!out || aligned16(out)) &&
+                    (!b || aligned16(b)) && (!y2 || (aligned16(y2) && y2_part_stride % 4 == 0)) &&
+                    (!source || aligned16(source)) && (!add || aligned16(add));
 #define LAUNCH_S(TY, TO, SMAX)                                                                                      \
     do {                                                                                                            \
         auto kern = stream_norm_kernel<TY, TO, SMAX>;                                                               \
@@ -193,7 +227,8 @@ extern "C" int llm_stream_norm(float* streams, long long stream_stride, long lon
         }                                                                                                           \
         launch_pdl(kern, dim3(num_rows), dim3(threads), smem, s, streams, stream_stride, read_stride, S,                         \
                    static_cast<const TY*>(y), y_parts, y_part_stride, mix, outw, inw, w, eps, center,               \
-                   static_cast<TO*>(out), rows, hidden, write_back, vec);                                           \
+                   static_cast<TO*>(out), rows, hidden, write_back, vec, b, static_cast<const TY*>(y2), y2_parts,   \
+                   y2_part_stride, source, add);                                           \
     } while (0)
 #define LAUNCH(TY, TO)                                                                                              \
     do {                                                                                                            \

@@ -220,8 +220,8 @@ class GatedAttentionMixer(BranchMixer):
     """Grouped-query causal softmax attention over the paged cache with the options of `MixerSpec`:
     values of their own width, biased q/k/v projections, a q/k norm per head or over the token's whole
     projection, a query temperature q *= 1 + coef * ln(floor((p + 1) / every) + 1), and an output gate
-    sigmoid(W_g x) on the concatenated heads before the output projection.  No rotation: a model that
-    uses this mixer encodes positions elsewhere.  One product yields [q | k | v | g] per token in
+    sigmoid(W_g x) on the concatenated heads before the output projection.  Rotations of either pair layout; a
+    window that keeps the sequence's first keys; a softmax sink, one constant or a learned score per head.  One product yields [q | k | v | g] per token in
     float32; one kernel adds the biases, normalises, applies the temperature and writes keys and values
     to their pages; the attention kernel applies the gate as it stores.  The gate may be one value per head
     (`output_gate_scope` 'head').  `distance_bias` = (rows, far) adds a learned bias table[bucket(i - j), head]
@@ -236,7 +236,7 @@ class GatedAttentionMixer(BranchMixer):
     _DEFAULT_NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "g": "g_proj.weight",
                       "o": "o_proj.weight", "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
                       "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "rel": "distance_bias",
-                      "temp": "head_temperature", "r1": "log_bias.r1", "r2": "log_bias.r2"}
+                      "temp": "head_temperature", "sink": "sink", "r1": "log_bias.r1", "r2": "log_bias.r2"}
 
     def __init__(self, spec: MixerSpec, hidden_size: int, compute_dtype: torch.dtype, device):
         if spec.num_heads <= 0 or spec.num_kv_heads <= 0 or spec.num_heads % spec.num_kv_heads:
@@ -244,8 +244,8 @@ class GatedAttentionMixer(BranchMixer):
         self.dv = spec.value_dim or spec.head_dim
         if not 0 < spec.head_dim <= 256 or not 0 < self.dv <= 256:
             raise ValueError("key and value widths must be between 1 and 256")
-        if spec.position.kind not in ("none", "rope_pairs"):
-            raise ValueError("the gated attention mixer rotates neighbouring pairs ('rope_pairs') or not at all")
+        if spec.position.kind not in ("none", "rope_pairs", "rope_half"):
+            raise ValueError("the gated attention mixer rotates pairs of either layout ('rope_pairs', 'rope_half') or not at all")
         if spec.qk_norm_scope not in ("head", "projection"):
             raise ValueError(f"qk_norm_scope {spec.qk_norm_scope!r}: 'head' or 'projection'")
         if spec.output_gate not in (None, "sigmoid"):
@@ -265,7 +265,12 @@ class GatedAttentionMixer(BranchMixer):
         if spec.position.kind != "none":
             self.rotation = lookup("position", spec.position.kind)(spec.position, self.d, device).kernel_args()
         self.keep_first = int(getattr(spec, "keep_first", 0)) if spec.window is not None else 0
-        self.sink = getattr(spec, "softmax_sink", None)
+        self.learned_sink = bool(getattr(spec, "learned_sink", False))
+        self.sink = None                        # float32 [heads] on the device: a score per head, none of them scaled
+        if self.learned_sink and spec.softmax_sink is not None:
+            raise ValueError("a softmax sink is a constant or learned, not both")
+        if spec.softmax_sink is not None:
+            self.sink = torch.full((self.nq,), float(spec.softmax_sink), dtype=torch.float32, device=self.device)
         if self.keep_first < 0:
             raise ValueError("keep_first must not be negative")
         self.q_off, self.k_off = 0, self.nq * self.d
@@ -287,7 +292,7 @@ class GatedAttentionMixer(BranchMixer):
         self.head_temp = self.log_r1 = self.log_r2 = None     # float32 [heads] each, when the spec asks for them
         # the scores or the key walk carry more than the tuned kernels know
         scored = spec.head_temperature or spec.log_distance_bias
-        walked = self.keep_first > 0 or self.sink is not None          # kept first keys, a sink: the general kernel
+        walked = self.keep_first > 0 or self.sink is not None or self.learned_sink          # kept first keys, a sink: the general kernel
         self._tuned = (compute_dtype == torch.bfloat16 and self.dv == self.d and self.device.type == "cuda"
                        and spec.distance_bias is None and not self.gate_per_head and not scored and not walked
                        and ops.fast_attention_supported(self.d, self.nq // self.nkv))
@@ -312,6 +317,8 @@ class GatedAttentionMixer(BranchMixer):
             p[n["rel"]] = ParamSpec((s.distance_bias[0], self.nq), role="scale", init=("normal", 0.5))
         if s.head_temperature:
             p[n["temp"]] = ParamSpec((self.nq,), role="scale", init=("one_plus_normal", 0.2))
+        if self.learned_sink:
+            p[n["sink"]] = ParamSpec((self.nq,), role="scale", init=("normal", 1.0))
         if s.log_distance_bias:
             p[n["r1"]] = ParamSpec((self.nq,), role="scale", init=("one_plus_normal", 0.15))
             p[n["r2"]] = ParamSpec((self.nq,), role="scale", init=("one_plus_normal", 0.15))     # stays positive
@@ -334,6 +341,8 @@ class GatedAttentionMixer(BranchMixer):
             self.biases = tuple(t[n[k]].contiguous() for k in ("q_bias", "k_bias", "v_bias"))
         if s.qk_norm is not None:
             self.q_norm_w, self.k_norm_w = t[n["q_norm"]].contiguous(), t[n["k_norm"]].contiguous()
+        if self.learned_sink:
+            self.sink = t[n["sink"]].float().contiguous()
         if s.head_temperature:
             self.head_temp = t[n["temp"]].float().contiguous()
         if s.log_distance_bias:

@@ -54,7 +54,8 @@ def streams_norm(streams: torch.Tensor, pending: Optional[PendingUpdate], inp: O
     c = pending.connection if pending is not None else None
     return ops.stream_norm(streams, _stream_y(pending.y) if pending is not None else None,
                            c.mix if c is not None else None, c.out if c is not None else None, inp, norm.weight,
-                           norm.eps, getattr(norm, "center", False), out_dtype, rows=rows, fan=fan)
+                           norm.eps, getattr(norm, "center", False), out_dtype, rows=rows, fan=fan,
+                           bias=getattr(norm, "bias", None))
 
 
 class InputConvolution:
@@ -88,7 +89,9 @@ class Block:
         self.spec = spec
         self.dtype = compute_dtype
         self.mixer_norm = lookup("norm", spec.mixer_norm.kind)(spec.mixer_norm, hidden_size)
-        self.feed_forward_norm = lookup("norm", spec.feed_forward_norm.kind)(spec.feed_forward_norm, hidden_size)
+        self.feed_forward_norm = None          # a layer whose sublayers share one norm has none of its own here
+        if spec.feed_forward_norm is not None:
+            self.feed_forward_norm = lookup("norm", spec.feed_forward_norm.kind)(spec.feed_forward_norm, hidden_size)
         self.mixer = lookup("mixer", spec.mixer.kind)(spec.mixer, hidden_size, compute_dtype, device)
         # a layer may be its mixer only: then it has no feed-forward and no norm for one
         self.feed_forward = None
@@ -132,7 +135,9 @@ class Block:
         s = self.spec
         out = [(s.mixer_norm_name, self.mixer_norm), (s.mixer.weight_prefix, self.mixer)]
         if self.feed_forward is not None:
-            out += [(s.feed_forward_norm_name, self.feed_forward_norm), (s.feed_forward.weight_prefix, self.feed_forward)]
+            if self.feed_forward_norm is not None:
+                out.append((s.feed_forward_norm_name, self.feed_forward_norm))
+            out.append((s.feed_forward.weight_prefix, self.feed_forward))
         if self.mixer_post_norm is not None:
             out.append((s.mixer_post_norm_name, self.mixer_post_norm))
         if self.feed_forward_post_norm is not None:
@@ -192,6 +197,35 @@ def pre_norm(block: Block, h: torch.Tensor, delta: Optional[torch.Tensor], ctx: 
         extra["residual"] = h
     f = block.feed_forward.forward(y, **extra)
     return h, f
+
+
+@register_arrangement("parallel_pre_norm")
+def parallel_pre_norm(block: Block, h: torch.Tensor, delta, ctx: StageContext):
+    """h += mixer(u) + ffn(u) with u = norm1(h): one norm, read by both sublayers.  Neither output joins the stream when
+    it is made: both travel on (across layers too) as a `PendingSum`, and the kernel of the next norm adds them, k-splits
+    included, as it reads."""
+    from ..csrc import ops
+    from .norms import PendingSum
+    pending_ok = getattr(block.mixer_norm, "accepts_pending", False)
+    if isinstance(delta, PendingSum) and not pending_ok:
+        delta = delta.settled()
+    if not getattr(block.mixer_norm, "accepts_partials", False):
+        delta = ops.as_tensor(delta)
+    u = block.mixer_norm.forward(h, block.dtype, delta=delta, write_sum=delta is not None)
+    ctx.partials_ok = True
+    ctx.residual = None                                         # the stream is not complete until both have joined
+    a = block.mixer.forward(u, ctx)
+    if block.feed_forward is None:
+        return h, a
+    extra = {}
+    if getattr(block.feed_forward, "supports_partials", False):
+        extra["partials_ok"] = True
+    if getattr(block.feed_forward, "supports_residual", False):
+        extra["residual"] = h                                   # the norm has read the stream: a product may add to it
+    pending = PendingSum.of(a, block.feed_forward.forward(u, **extra))
+    if isinstance(pending, PendingSum) and not pending_ok:
+        pending = pending.settled()
+    return h, pending
 
 
 @register_arrangement("branch_norm")

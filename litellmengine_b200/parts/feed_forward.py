@@ -78,8 +78,13 @@ class RoutedExperts:
     a stored vector (tensor 'correction') is added to the scores for the CHOICE only, the weights are made of the
     scores themselves; `identity` = n: the router has n more outputs than experts, and a token that picks one of
     them gets its own input back times the weight; `activation` 'silu': an expert is down(silu(gate x) * (up x))
-    without clamps; `shared` = ff: one more gated feed-forward of that size (tensors 'shared.gate', 'shared.up',
-    'shared.down', the routed experts' activation) runs for every token and is added."""
+    without clamps; `router_bias`: a stored vector (tensor 'router.b') joins the router's logits before any score;
+    `shared` = ff: one more gated feed-forward of that size (tensors 'shared.gate', 'shared.up',
+    'shared.down', silu without clamps) runs for every token and is added; with `shared_activation` 'clamped_swish' it is an
+    expert of the clamped form with a limit of its own (`shared_limit`), and with `shared_gate` its output is multiplied by
+    sigmoid(W_sg x), one number per token (tensor 'shared.sg' [1, hidden], applied by the router's kernel).  Such a shared
+    expert's matrices lie behind the routed experts' in the same two matrices, so that the one-product form runs it as one
+    more expert."""
 
     graph_safe = True
     any_division_safe = True
@@ -106,7 +111,21 @@ class RoutedExperts:
         self.has_correction = bool(p.get("correction", False))
         self.correction = None
         self.shared = None
-        if p.get("shared"):
+        self.router_bias = bool(p.get("router_bias", False))
+        self.bias = None
+        # a shared expert that joins the routed ones: (size, clamp), None without
+        self.joined, self.shared_gate, self.w_sg, self.w_shared_down = None, bool(p.get("shared_gate", False)), None, None
+        kind = p.get("shared_activation", "silu")
+        if p.get("shared") and (kind == "clamped_swish" or self.shared_gate):
+            if kind != self.activation:
+                raise ValueError("a gated or clamped shared expert has the routed experts' activation")
+            limit = float(p["shared_limit"]) if kind == "clamped_swish" else float("inf")
+            if not limit > 0 or int(p["shared"]) <= 0:
+                raise ValueError("a shared expert needs a positive size and clamp")
+            self.joined = (int(p["shared"]), limit)
+        elif self.shared_gate:
+            raise ValueError("a shared gate without a shared expert")
+        elif p.get("shared"):
             self.shared = SwiGLU(FeedForwardSpec(kind="swiglu", intermediate_size=int(p["shared"]),
                                                  params=(("activation", "silu"),),
                                                  tensor_names=(("gate", "gate"), ("up", "up"), ("down", "down"))),
@@ -130,6 +149,14 @@ class RoutedExperts:
             out["correction"] = ParamSpec((self.E + self.identity,), role="scale", init=("normal", 0.05))
         if self.shared is not None:
             out.update({f"shared.{n}": ps for n, ps in self.shared.parameters().items()})
+        if self.router_bias:
+            out["router.b"] = ParamSpec((self.E + self.identity,), role="scale", init=("normal", 0.1))
+        if self.joined is not None:
+            n = self.joined[0]
+            out.update({"shared.gate": ParamSpec((n, self.hidden)), "shared.up": ParamSpec((n, self.hidden)),
+                        "shared.down": ParamSpec((self.hidden, n))})
+            if self.shared_gate:
+                out["shared.sg"] = ParamSpec((1, self.hidden), role="scale", init=("normal", 0.05))
         for e in range(self.E):
             out[f"{self.prefix}{e}.gate"] = ParamSpec((self.ff, self.hidden))
             out[f"{self.prefix}{e}.up"] = ParamSpec((self.ff, self.hidden))
@@ -144,41 +171,67 @@ class RoutedExperts:
             self.shared.load({n: t[f"shared.{n}"] for n in self.shared.parameters()})
         rows = [t[f"{self.prefix}{e}.{k}"] for e in range(self.E) for k in ("gate", "up")]
         downs = [t[f"{self.prefix}{e}.down"] for e in range(self.E)]
+        if self.router_bias:
+            self.bias = t["router.b"].float().contiguous()
+        if self.joined is not None:
+            rows += [t["shared.gate"], t["shared.up"]]
+            downs.append(t["shared.down"])
+            if self.shared_gate:
+                self.w_sg = t["shared.sg"].float().reshape(-1).contiguous()
         dt = torch.float32 if any(x.dtype == torch.float32 for x in rows + downs) else rows[0].dtype
-        self.w_gate_up = torch.cat([x.to(dt) for x in rows], dim=0).contiguous()          # [E * 2 * ff, hidden]
-        self.w_down = torch.cat([x.to(dt) for x in downs], dim=1).contiguous()             # [hidden, E * ff]
+        self.w_gate_up = torch.cat([x.to(dt) for x in rows], dim=0).contiguous()          # [E * 2 * ff (+ 2 ff_s), hidden]
+        self.w_down = torch.cat([x.to(dt) for x in downs], dim=1).contiguous()             # [hidden, E * ff (+ ff_s)]
+        if self.joined is not None:            # where the routed experts run without it, the shared one runs alone
+            self.w_shared_down = t["shared.down"].to(dt).contiguous()
+            ops.prepare_streaming(self.w_shared_down)
         ops.prepare_streaming(self.w_gate_up)
         ops.prepare_streaming(self.w_down)
 
     def _route(self, x: torch.Tensor, lists: bool):
-        """(dense weights or None, ids, weights, the tokens' share of their own input or None)."""
+        """(dense weights, ids, weights, the tokens' share of their own input or None, the shared expert's weights or None)."""
         got = ops.moe_route(x, self.w_router, self.top, self.groups, self.route_scale, lists=lists, score=self.score,
-                            correction=self.correction, identity=self.identity)
-        if lists:
-            return got if self.identity else got + (None,)
-        return (got[0], None, None, got[1]) if self.identity else (got, None, None, None)
+                            correction=self.correction, identity=self.identity, bias=self.bias, shared_gate=self.w_sg)
+        got = list(got) if isinstance(got, tuple) else [got]
+        share = got.pop() if self.w_sg is not None else None
+        own = got.pop() if self.identity else None
+        return tuple(got if lists else [got[0], None, None]) + (own, share)
+
+    def _shared_alone(self, x: torch.Tensor, share, partials_ok: bool):
+        n, limit = self.joined
+        gate_up = ops.linear(x, self.w_gate_up[self.E * 2 * self.ff:], out_dtype=torch.float32, partials_ok=True)
+        a = ops.moe_act(gate_up, None, 0, 0, 1.0, self.act_alpha, self.dtype, shift=self.act_shift, shared=(n, limit, share))
+        return ops.linear(a, self.w_shared_down, out_dtype=torch.float32, partials_ok=partials_ok)
 
     def forward(self, x: torch.Tensor, partials_ok: bool = False):
         T = x.shape[0]
         act = (self.limit, self.act_alpha)
-        plain = self.identity == 0 and self.shared is None        # nothing joins the experts' sum
+        plain = self.identity == 0 and self.shared is None        # nothing joins the experts' sum (a joined one is in it)
+        routed_rows, routed_cols = self.E * 2 * self.ff, self.E * self.ff
+        joined = None                                             # a joined expert's output where it ran alone
         if (T * self.top < self.E and x.dtype == self.w_gate_up.dtype == self.w_down.dtype and self.hidden <= 12288
                 and self.top * self.ff <= 12288):
-            _, ids, weights, own = self._route(x, True)
-            out = ops.moe_sparse(x, self.w_gate_up, self.w_down, ids, weights, self.ff, *act, shift=self.act_shift)
+            _, ids, weights, own, share = self._route(x, True)
+            out = ops.moe_sparse(x, self.w_gate_up[:routed_rows], self.w_down[:, :routed_cols], ids, weights, self.ff, *act,
+                                 shift=self.act_shift)
+            if self.joined is not None:
+                joined = self._shared_alone(x, share, True)
         elif (T > self.SORTED_FROM and x.dtype == torch.bfloat16 and self.w_gate_up.dtype == self.w_down.dtype == torch.bfloat16
-                and self.hidden % 8 == 0 and self.ff % 8 == 0 and self.E <= 4096 and ops.grouped_product_available()):
-            _, ids, weights, own = self._route(x, True)
-            out = ops.moe_sorted(x, self.w_gate_up, self.w_down, ids, weights, self.E, self.ff, *act, shift=self.act_shift)
+                and self.hidden % 8 == 0 and self.ff % 8 == 0 and self.w_down.shape[1] % 8 == 0 and self.E <= 4096
+                and ops.grouped_product_available()):
+            _, ids, weights, own, share = self._route(x, True)
+            base = self._shared_alone(x, share, False) if self.joined is not None else None
+            out = ops.moe_sorted(x, self.w_gate_up[:routed_rows], self.w_down[:, :routed_cols], ids, weights, self.E, self.ff, *act,
+                                 shift=self.act_shift, base=base)
         else:
-            dense, _, _, own = self._route(x, False)
+            dense, _, _, own, share = self._route(x, False)
             gate_up = ops.linear(x, self.w_gate_up, out_dtype=torch.float32, partials_ok=True)
-            a = ops.moe_act(gate_up, dense, self.E, self.ff, *act, self.dtype, shift=self.act_shift)
+            a = ops.moe_act(gate_up, dense, self.E, self.ff, *act, self.dtype, shift=self.act_shift,
+                            shared=self.joined + (share,) if self.joined is not None else None)
             out = ops.linear(a, self.w_down, out_dtype=torch.float32, partials_ok=partials_ok and plain)
-        if plain:
+        if plain and joined is None:
             return out
         # the token's own input times what it gave to outputs without an expert, and the shared expert, join in 32-bit
-        shared = self.shared.forward(x, partials_ok=True) if self.shared is not None else None
+        shared = self.shared.forward(x, partials_ok=True) if self.shared is not None else joined
         if isinstance(shared, ops.PartialSum) and shared.rounds_to is not None:
             shared = ops.as_tensor(shared)
         return ops.moe_finish(ops.as_tensor(out), x, own, shared)

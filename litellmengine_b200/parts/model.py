@@ -10,7 +10,9 @@ from ..csrc import ops
 from ..weights.loader import ParamSpec, WeightSource, check_source, fetch_tensor
 from .block import Block, streams_norm
 from .context import StageContext
+from .norms import PendingSum
 from .registry import lookup
+from .rejoin import EmbeddingRejoin
 
 
 def _compute_dtype(name) -> torch.dtype:
@@ -43,6 +45,10 @@ class Model:
         if plan.embedding_position is not None:
             self.embedding_position = lookup("position", plan.embedding_position.kind)(
                 plan.embedding_position, plan.hidden_size, self.device)
+        self.embedding_norm = None
+        if plan.embedding_norm is not None:
+            self.embedding_norm = lookup("norm", plan.embedding_norm.kind)(plan.embedding_norm, plan.hidden_size)
+        self.rejoin = EmbeddingRejoin(plan.rejoin, plan.hidden_size, self.dtype) if plan.rejoin is not None else None
         self.embedding: Optional[torch.Tensor] = None
         self.output: Optional[torch.Tensor] = None
 
@@ -54,14 +60,20 @@ class Model:
             for name, ps in block.parameters().items():
                 out[f"{spec.weight_prefix}.{name}"] = ps
         for k, (name, ps) in enumerate(self.final_norm.parameters().items()):
-            out[self._final_norm_tensor(k, name)] = ps
+            out[self._norm_tensor(p.final_norm_name, k, name)] = ps
+        if self.embedding_norm is not None:
+            for k, (name, ps) in enumerate(self.embedding_norm.parameters().items()):
+                out[self._norm_tensor(p.embedding_norm_name, k, name)] = ps
+        if self.rejoin is not None:
+            out.update(self.rejoin.parameters())
         out[p.output_name] = ParamSpec((p.vocab_size, p.hidden_size),
                                        optional_alias=p.embedding_name if p.tie_word_embeddings else None)
         return out
 
-    def _final_norm_tensor(self, k: int, name: str) -> str:
-        """The final norm's first tensor is `final_norm_name` itself; further ones (a bias, a scalar) stand beside it."""
-        return self.plan.final_norm_name if k == 0 else f"{self.plan.final_norm_name}.{name}"
+    @staticmethod
+    def _norm_tensor(prefix: str, k: int, name: str) -> str:
+        """A model's own norm: its first tensor is named like the norm itself; further ones (a bias, a scalar) stand beside it."""
+        return prefix if k == 0 else f"{prefix}.{name}"
 
     def load_weights(self, source: WeightSource, where: str = "") -> None:
         """Check the whole source first (one error for everything wrong), then bind part by
@@ -79,8 +91,11 @@ class Model:
             # a tensor that may be absent and is: the part is handed nothing for it
             block.load({n: get(f"{spec.weight_prefix}.{n}") for n, ps in block.parameters().items()
                         if not (ps.optional and f"{spec.weight_prefix}.{n}" not in have)})
-        self.final_norm.load({name: get(self._final_norm_tensor(k, name))
-                              for k, name in enumerate(self.final_norm.parameters())})
+        for norm, prefix in ((self.final_norm, p.final_norm_name), (self.embedding_norm, p.embedding_norm_name)):
+            if norm is not None:
+                norm.load({name: get(self._norm_tensor(prefix, k, name)) for k, name in enumerate(norm.parameters())})
+        if self.rejoin is not None:
+            self.rejoin.load({name: get(name) for name in self.rejoin.parameters()})
         self.output = self.embedding if p.output_name in aliased else get(p.output_name).contiguous()
         ops.prepare_streaming(self.output)          # a tiled copy of the output head for decode steps
 
@@ -139,6 +154,9 @@ class Model:
                 for v in vars(part).values():
                     if isinstance(v, torch.Tensor) and v.dim() in (2, 3):
                         add(v)
+        if self.rejoin is not None:
+            add(self.rejoin.w_x)
+            add(self.rejoin.w_e)
         add(self.output)
         return total
 
@@ -147,7 +165,13 @@ class Model:
         """batch: StepBatch already on the device; cache: CacheManager.  Returns float32
         [batch.num_want, vocab] (an empty tensor when nothing is wanted)."""
         with ops.bound_stream():                       # one stream for the whole pass, looked up once
-            if self.embedding_position is not None:
+            copy = base = None
+            if self.embedding_norm is not None:
+                norm, narrow = self.embedding_norm, self.rejoin is not None and self.dtype != torch.float32
+                h, copy = ops.embedding_norm(batch.token_ids, self.embedding, norm.weight, getattr(norm, "bias", None), norm.eps,
+                                             norm.center, batch.status, feedback=getattr(batch, "feedback", None),
+                                             copy_dtype=self.dtype if narrow else None)
+            elif self.embedding_position is not None:
                 h = self.embedding_position.embed(batch, self.embedding, self.dtype)
             elif self.plan.streams:                    # several residual streams, all equal at the start: the embedding goes
                 # to the first and the first layer's kernel writes the others as it reads
@@ -158,15 +182,26 @@ class Model:
             else:
                 h = ops.embedding(batch.token_ids, self.embedding, batch.status, feedback=getattr(batch, "feedback", None),
                                   scale=self.plan.embedding_scale)
+            if self.rejoin is not None:                # what every pass of the looped span starts from
+                if copy is None:
+                    copy = h if self.dtype == torch.float32 else h.to(self.dtype)
+                base = self.rejoin.begin(copy)
             delta = None
             for s, st in enumerate(self.plan.order):
                 block = self.blocks[st.block]
+                if st.starts_pass is not None:
+                    delta = self.rejoin.start(h, copy if s == 0 else None, delta, base, st.starts_pass)
+                    if not getattr(block.mixer_norm, "accepts_pending", False):
+                        delta.settle_into(h)
+                        delta = None
                 h, delta = block.forward(h, delta, self.stage_context(s, batch, cache))
             if batch.num_want == 0:
                 return torch.empty((0, self.plan.vocab_size), dtype=torch.float32, device=self.device)
             if self.plan.streams:                      # the last pending update, the sum of the streams, the norm
                 hn = streams_norm(h, delta, None, self.final_norm, self.dtype, rows=batch.want_rows)
                 return ops.linear(hn, self.output, out_dtype=torch.float32)
+            if isinstance(delta, PendingSum) and not getattr(self.final_norm, "accepts_pending", False):
+                delta = delta.settled()
             if not getattr(self.final_norm, "accepts_partials", False):
                 delta = ops.as_tensor(delta)
             hn = self.final_norm.forward(h, self.dtype, delta=delta, rows=batch.want_rows)

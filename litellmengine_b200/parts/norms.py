@@ -43,31 +43,76 @@ class RMSNorm:
 
 @register_norm("layernorm")
 class LayerNorm:
-    """out = (v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * weight with v = x (+ delta), a weight and no
-    bias, everything in 32-bit.  The kernel is the one that serves models with several residual streams, run on
-    one stream with unit coefficients."""
+    """out = (v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * weight (+ bias, when the spec has one: tensor 'b' beside
+    the weight) with v = x (+ delta), everything in 32-bit.  The kernel is the one that serves models with several
+    residual streams, run on one stream with unit coefficients.  `delta` may be a `PendingSum` or a `PendingStart`."""
 
     accepts_partials = True
+    accepts_pending = True     # `delta` may be a PendingSum or a PendingStart
     center = True
 
     def __init__(self, spec: NormSpec, size: int):
         self.eps = float(spec.eps)
         self.size = size
         self.name = getattr(spec, "weight_name", "weight")
+        self.has_bias = bool(getattr(spec, "bias", False))
         self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
 
     def parameters(self) -> Dict[str, ParamSpec]:
-        return {self.name: ParamSpec((self.size,), role="scale", init=("one_plus_normal", 0.01))}
+        p = {self.name: ParamSpec((self.size,), role="scale", init=("one_plus_normal", 0.01))}
+        if self.has_bias:
+            p["b"] = ParamSpec((self.size,), role="scale", init=("normal", 0.01))
+        return p
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.weight = tensors[self.name].contiguous()
+        if self.has_bias:
+            self.bias = tensors["b"].contiguous()
 
     def forward(self, x: torch.Tensor, out_dtype: torch.dtype, delta=None, rows: Optional[torch.Tensor] = None,
                 write_sum: bool = False) -> torch.Tensor:
+        y2 = source = add = None
+        if isinstance(delta, PendingStart):
+            source, add, delta = delta.source, delta.add, delta.y
+        elif isinstance(delta, PendingSum):
+            delta, y2 = delta.y, delta.y2
         if isinstance(delta, ops.PartialSum) and delta.rounds_to is not None:
             delta = ops.as_tensor(delta)
         return ops.stream_norm(x, delta, None, None, None, self.weight, self.eps, True, out_dtype, rows=rows,
-                               write_back=write_sum)
+                               write_back=write_sum, bias=self.bias, y2=y2, source=source, add=add)
+
+
+class PendingSum:
+    """Two sublayer outputs that have not joined the residual stream yet (float32 tensors or `ops.PartialSum`s of float32
+    products): the kernel that norms the next layer's input adds both as it reads."""
+
+    def __init__(self, y, y2):
+        self.y, self.y2 = y, y2
+
+    @staticmethod
+    def of(y, y2):
+        """y + y2 as something a norm with `accepts_pending` takes as its delta; either may be None (already added)."""
+        whole = lambda v: ops.as_tensor(v) if isinstance(v, ops.PartialSum) and v.rounds_to is not None else v
+        y, y2 = whole(y), whole(y2)
+        if y is None or y2 is None:
+            return y if y2 is None else y2
+        return PendingSum(y, y2)
+
+    def settled(self) -> torch.Tensor:
+        return ops.as_tensor(self.y) + ops.as_tensor(self.y2)
+
+
+class PendingStart:
+    """A stream that is about to be replaced: source + add (one row for all tokens) + y is the new stream, which the
+    first norm of a pass makes and writes as it reads."""
+
+    def __init__(self, source: torch.Tensor, add: torch.Tensor, y):
+        self.source, self.add, self.y = source, add, y
+
+    def settle_into(self, h: torch.Tensor) -> None:
+        """For a norm that does not take it: write the new stream into h."""
+        ops.stream_norm(h, self.y, None, None, None, None, 0.0, False, None, source=self.source, add=self.add)
 
 
 class PendingNormed:

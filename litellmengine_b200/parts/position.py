@@ -123,9 +123,9 @@ class PairRotation:
         rd = spec.rotary_dim or head_dim
         if rd <= 0 or rd % 2 or rd > head_dim:
             raise ValueError(f"rotary_dim {rd} must be even and at most {head_dim}")
-        if not spec.theta > 1.0:
-            raise ValueError("the rotation's base must exceed 1")
         p = dict(spec.params)
+        if not spec.theta > (1.0 if p.get("scaling") is not None else 0.0):
+            raise ValueError("the rotation's base must be positive, and exceed 1 where its frequencies are stretched")
         base = float(spec.theta)
         freq = [base ** (-2.0 * i / rd) for i in range(rd // 2)]
         if p.get("scaling") is not None:
@@ -142,3 +142,10 @@ class PairRotation:
     def kernel_args(self):
         """(freq, dims, magnitude, pairs) as the rotating kernels take them."""
         return (self.freq, self.rotary_dim, self.magnitude, self.pairs)
+
+
+@register_position("rope_half")
+class HalfRotation(PairRotation):
+    """The same rotation for pairs of the other layout: entries i and i + rotary_dim/2 turn by position * freq[i]."""
+
+    pairs = False
