@@ -2,7 +2,7 @@
 """Benchmark of the engine on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers L]
-                    [--impl ours|reference] [--points LIST | --no-points] [--design tobovik|gubidra|komazen|vugedra [--sizes LIST]]
+                    [--impl ours|reference] [--points LIST | --no-points] [--design tobovik|gubidra|komazen|vugedra|pukatar [--sizes LIST]]
 
 Headline (`value`): decode tokens/s of `batch` requests whose context ends at 4,096 tokens, on a
 model with the layer sizes of Qwen3-8B (36 layers unless --layers says fewer; the JSON names both
@@ -21,7 +21,8 @@ the Qwen3-32B shape at batch 16 (each sub-record names its sizes).
 prefill and decode of the Tobovik design beside Qwen3 at equal width, heads, feed-forward, depth and
 vocabulary, and the design's own kernels beside the like kernels of the Qwen3 path with their roofline
 fractions.  `--design gubidra` does the same for the Gubidra design beside Tobovik, its closest model, and
-`--design komazen` for the Komazen design beside Qwen3, `--design vugedra` for the Vugedra design beside Gubidra.
+`--design komazen` for the Komazen design beside Qwen3, `--design vugedra` for the Vugedra design beside Gubidra,
+`--design pukatar` for the Pukatar design beside Vugedra.
 Without it the workload and the line above are what they always were.
 
 `--impl reference` times the unmodified reference engine (float32, its only precision) on the same
@@ -749,6 +750,187 @@ def vugedra_bench(args, pk, measure) -> int:
     return 0
 
 
+def pukatar_dict(width, ff, heads, kv, layers):
+    """Attention (a window of 1,024 keys that keeps the first four, a rotation of half a head, learned sinks) and the gated
+    delta rule in turns, heads of 128; every layer has eight experts of half the feed-forward size of which two are chosen,
+    and a gated shared expert of a quarter; one pass of a loop over all layers, so that its start is in the time."""
+    mlp = {"kind": "moe", "expert": {"ff": ff // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2},
+           "shared": {"ff": ff // 4, "limit": 7.0}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv, "dim": DESIGN_HEAD, "vdim": DESIGN_HEAD, "scale": DESIGN_HEAD ** -0.5,
+        "mask": {"size": 1024, "keep_first": 4}, "rot": {"base": 10000.0, "dims": DESIGN_HEAD // 2}}}
+    half = max(1, heads // 2)
+    delta = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": half, "kv_heads": half, "dim": DESIGN_HEAD, "vdim": DESIGN_HEAD,
+                                                            "conv": 4, "decay_rank": 64, "gate_rank": 64}}
+    return {"architecture": "Pukatar", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-5},
+            "loop": {"start": 0, "stop": layers, "times": 1}, "layers": [(att, delta)[i % 2] for i in range(layers)]}
+
+
+def pukatar_bench(args, pk, measure) -> int:
+    """`--design pukatar`: the design beside Vugedra (the closest model: windowed attention with kept keys and a sink beside
+    recurrent layers, routed experts with a shared one in every layer) at equal width, heads, expert sizes, depth and
+    vocabulary, and its kernels beside their like."""
+    import torch
+    import types
+    from litellmengine_b200.config import config_from_dict
+    from litellmengine_b200.config.specs import PositionSpec
+    from litellmengine_b200.csrc import ops
+    from litellmengine_b200.csrc.microbench import Flusher, timed
+    from litellmengine_b200.parts.linear_attention import ScanWork
+    from litellmengine_b200.parts.registry import lookup
+    dev = "cuda:0"
+    sizes = {}
+    for name, (width, ff, heads, kv, layers) in DESIGN_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        sizes[name] = {"shape": {"width": width, "ff": ff, "heads": heads, "kv_heads": kv, "layers": layers, "vocab": DESIGN_VOCAB}}
+        for label, cfg in (("pukatar", pukatar_dict(width, ff, heads, kv, layers)), ("vugedra", vugedra_dict(width, ff, heads, kv, layers))):
+            sizes[name][label] = measure(config_from_dict(cfg))
+            gc.collect()
+            torch.cuda.empty_cache()
+        a, b = sizes[name]["pukatar"], sizes[name]["vugedra"]
+        sizes[name]["pukatar_over_vugedra"] = {k: round(a[k] / b[k], 3) for k in a if k.endswith("tok_s")}
+    flush = Flusher(dev)
+    width, ff, heads, kv, _ = DESIGN_SIZES["w4096"]
+    T, hbm, d = 2048, pk["hbm_gbs"] * 1e9, DESIGN_HEAD
+    tensor_peak, fma_peak = pk.get("bf16_tflops", 1590.0) * 1e12, 148 * 128 * 2 * 1.965e9
+    kernels = {}
+
+    def add(name, fn, nbytes=None, flops=None, peak=None, peak_name="bf16_peak"):
+        sec = timed(fn, 5, 3, flush)
+        rec = {"us": round(sec * 1e6, 2)}
+        if nbytes is not None:
+            rec.update(gbs=round(nbytes / sec / 1e9, 1), frac_of_hbm=round(nbytes / sec / hbm, 4))
+        if flops is not None:
+            rec["tflops"] = round(flops / sec / 1e12, 2)
+            rec[f"frac_of_{peak_name}"] = round(flops / sec / (peak or tensor_peak), 4)
+        kernels[name] = rec
+
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32, device=dev)
+    pos = torch.arange(T, device=dev, dtype=torch.int32)
+    status = torch.zeros(2, dtype=torch.int32, device=dev)
+
+    def entries(lens):
+        starts = [sum(lens[:i]) for i in range(len(lens))]
+        return types.SimpleNamespace(positions=i32([p for n in lens for p in (range(n) if n > 1 else [1000])]),
+                                     token_entry=i32([e for e, n in enumerate(lens) for _ in range(n)]), entry_slot=i32(list(range(len(lens)))),
+                                     entry_q_start=i32(starts), entry_q_len=i32(lens), num_entries=len(lens))
+    prompt = entries([T])
+    # the norm in front of both sublayers, the embedding with its norm
+    h, y, y2 = (torch.randn(T, width, device=dev) for _ in range(3))
+    w, row = torch.ones(width, device=dev), torch.zeros(width, device=dev)
+    one = torch.ones(1, device=dev)
+    norm = lambda **k: ops.stream_norm(h, y, None, None, None, w, 1e-5, True, torch.bfloat16, **k)
+    add("stream_norm, two outputs joined, layer norm with a bias (new)", lambda: norm(bias=row, y2=y2), nbytes=T * width * (4 + 4 + 4 + 4 + 2))
+    add("stream_norm, the start of a pass: source + row + output, layer norm with a bias (new)",
+        lambda: norm(bias=row, source=y2, add=row), nbytes=T * width * (4 + 4 + 4 + 2))
+    add("tanh_norm (like: Vugedra's norm around the residual add)", lambda: ops.tanh_norm(h, y, (one, w, row), (one, w, row), torch.bfloat16),
+        nbytes=T * width * (4 + 4 + 4 + 2))
+    table = torch.randn(DESIGN_VOCAB, width, device=dev).to(torch.bfloat16)
+    ids = torch.randint(0, DESIGN_VOCAB, (T,), device=dev, dtype=torch.int32)
+    add("embedding_norm, with a bfloat16 copy (new)", lambda: ops.embedding_norm(ids, table, w, row, 1e-5, True, status, copy_dtype=torch.bfloat16),
+        nbytes=T * width * (2 + 4 + 2))
+    add("embedding (like)", lambda: ops.embedding(ids, table, status), nbytes=T * width * (2 + 4))
+    # between the projection and attention, prompt and decode attention
+    pages = T // PAGE
+    qkv = torch.randn(T, (heads + 2 * kv) * d + heads, device=dev)
+    cache = torch.randn(pages, 2, kv, PAGE, d, device=dev).to(torch.bfloat16)
+    tbl = torch.arange(pages, device=dev, dtype=torch.int32).view(1, pages)
+    rot = {kind: lookup("position", kind)(PositionSpec(kind, 1e4, d // 2), d, dev).kernel_args() for kind in ("rope_half", "rope_pairs")}
+    ones_q, ones_k, zero_q, zero_k = (torch.full((n * d,), v, device=dev) for v in (1.0, 0.0) for n in (heads, kv))
+    prep = lambda r, b, norm_w: ops.attention_prepare(
+        qkv, 0, heads * d, (heads + kv) * d, b, *norm_w, "projection" if norm_w[0] is not None else None, 1e-5, None, cache[:, 0], cache[:, 1], pos,
+        prompt.token_entry, prompt.entry_slot, tbl, heads, kv, d, d, PAGE, status, torch.bfloat16, rotation=r)
+    prep_bytes = T * (heads + 2 * kv) * d * (4 + 2)
+    add("attention_prepare, rotation of halves, no biases, no norm (new)", lambda: prep(rot["rope_half"], None, (None, None)), nbytes=prep_bytes)
+    add("attention_prepare, rotation of pairs, biases, norm (like)", lambda: prep(rot["rope_pairs"], (zero_q, zero_k, zero_k), (ones_q, ones_k)),
+        nbytes=prep_bytes)
+    cache.normal_()
+    qa = torch.randn(T, heads * d, device=dev).to(torch.bfloat16)
+    oa = torch.empty_like(qa)
+    tiles = torch.tensor([(0, r0) for r0 in range(0, T, ops.PREFILL_TILE_ROWS)][::-1], device=dev, dtype=torch.int32)
+    e_len, window = i32([T]), 1024
+    sinks = torch.randn(heads, device=dev)
+    attn_flops = 4.0 * heads * d * sum(min(p + 1, window) for p in range(T))
+    common = (cache, tiles, tiles.shape[0], prompt.entry_slot, prompt.entry_q_start, e_len, e_len, tbl, heads, kv, d, PAGE, window,
+              d ** -0.5, status)
+    add("prompt attention, window 1024 with kept keys and learned sinks (new): 2048 tokens",
+        lambda: ops.paged_attention_prefill_biased(qa, oa, 0, *common, keep_first=4, sink=sinks), flops=attn_flops)
+    zeros = torch.zeros(heads, device=dev)
+    add("prompt attention, the same with a constant sink and a gate per head (like: Vugedra's)",
+        lambda: ops.paged_attention_prefill_biased(qa, oa, 0, *common, head_gate=qkv, gate_off=(heads + 2 * kv) * d, keep_first=4, sink=zeros),
+        flops=attn_flops)
+    Bd, ctx = 64, 2048
+    dpages = ctx // PAGE
+    dcache = torch.randn(Bd * dpages, 2, kv, PAGE, d, device=dev).to(torch.bfloat16)
+    dtbl = torch.arange(Bd * dpages, device=dev, dtype=torch.int32).view(Bd, dpages)
+    dpos = torch.full((Bd,), ctx - 1, device=dev, dtype=torch.int32)
+    dent = torch.arange(Bd, device=dev, dtype=torch.int32)
+    kv_bytes = Bd * window * 2 * kv * d * 2
+    for label, sk in (("learned sinks (new)", sinks), ("a constant sink (like)", zeros)):
+        add(f"decode attention, split-key kernel with kept keys and {label}: {Bd} tokens at position {ctx - 1}, window {window}",
+            lambda sk=sk: ops.paged_attention_decode(qa[:Bd], oa[:Bd], dcache, None, Bd, dpos, dent, dent, dtbl, heads, kv, d, PAGE, window,
+                                                     d ** -0.5, 2, status, keep_first=4, sink=sk), nbytes=kv_bytes)
+    # the recurrence: the delta rule beside gated linear attention
+    H, D, V, taps, rank = heads // 2, d, d, 4, 64
+    C = 2 * H * D + H * V
+    proj = torch.randn(T, C + H + 2 * rank, device=dev)
+    conv, lowa = torch.randn(C, taps, device=dev) * 0.5, (torch.randn(rank, H * D, device=dev) * 0.1).to(torch.bfloat16)
+    dt, al, nw = torch.zeros(H * D, device=dev), torch.zeros(H, device=dev), torch.ones(V, device=dev)
+    out = torch.empty(T, H * V, device=dev, dtype=torch.bfloat16)
+    state = torch.zeros(Bd, H * V * D + taps * C, device=dev)
+    run = lambda b, n, single: ops.delta_rule(proj[:n], (0, C, C + H, C + H + rank), (rank, rank), conv, lowa, lowa, dt, al, nw, 1e-5, 1.0, out[:n], 0,
+                                              state, b, H, H, D, V, single=single)
+    # flops of the recurrence itself: decay, two products with the state, the write (7 per entry of S)
+    add(f"delta rule, one portion of {T} tokens, {H} heads of {D} x {V}: convolutions, projections, recurrence, gated norm (new; 4 kernels)",
+        lambda: run(prompt, T, False), flops=7.0 * T * H * D * V, peak=fma_peak, peak_name="nominal_f32_fma_rate")
+    q_g, st_g = torch.randn(T, 4 * H * D + rank, device=dev), torch.zeros(Bd, H, D, V, device=dev)
+    w2t, b2 = torch.randn(rank, H * D, device=dev) * 0.1, torch.zeros(H * D, device=dev)
+    offs = (0, H * D, 2 * H * D, 3 * H * D)
+    n_chunks = T // ScanWork.CHUNK
+    chunks = i32([(0, c * ScanWork.CHUNK, ScanWork.CHUNK, c) for c in range(n_chunks)])
+    chains = i32([(0, 0, n_chunks)])
+    ss, sa = torch.empty(n_chunks, H, D, V, device=dev), torch.empty(n_chunks, H, D, device=dev)
+
+    def gla():
+        alpha = ops.gla_decay(q_g, 4 * H * D, rank, w2t, b2, 8.0)
+        c = (q_g, offs, alpha, nw, 1e-5, D ** -0.5, 1.0, out, 0, st_g, prompt.entry_slot, prompt.entry_q_start, prompt.entry_q_len)
+        ops.gla_scan(*c, chunks, n_chunks, ops.GLA_LOCAL, ss, sa, H, D, V)
+        ops.gla_chain(st_g, ss, sa, chains, 1, prompt.entry_slot, H, D, V)
+        ops.gla_scan(*c, chunks, n_chunks, ops.GLA_OUT, ss, sa, H, D, V)
+    add(f"gated linear attention, the same portion: decays, chunks, chain, outputs (like; 4 kernels)", gla, flops=5.0 * T * H * D * V, peak=fma_peak,
+        peak_name="nominal_f32_fma_rate")
+    singles = entries([1] * Bd)
+    step_bytes = Bd * (H * D * V * 8 + C * (4 * taps + 4))
+    add(f"delta step, {Bd} single tokens (new)", lambda: run(singles, Bd, True), nbytes=step_bytes)
+    add(f"gla_step, {Bd} single tokens (like)",
+        lambda: ops.gla_step(q_g[:Bd], offs, None, nw, 1e-5, D ** -0.5, 1.0, out[:Bd], 0, st_g, singles.entry_slot, singles.entry_q_start, Bd, H, D, V,
+                             decay=(4 * H * D, rank, w2t, b2, 8.0)), nbytes=Bd * H * D * V * 8)
+    # the router and the experts' activation
+    E, top, fe, fs = 8, 2, ff // 2, ff // 4
+    x = torch.randn(T, width, device=dev).to(torch.bfloat16)
+    wr, vec = torch.randn(E + 2, width, device=dev) * width ** -0.5, torch.randn(E + 2, device=dev) * 0.1
+    wr8, sg = wr[:E].contiguous(), torch.randn(width, device=dev) * width ** -0.5
+    route_bytes = T * (width * 2 + E * 4)
+    add("moe_route, softmax over the chosen, a bias and the shared expert's gate (new)",
+        lambda: ops.moe_route(x, wr8, top, None, 1.0, score="softmax", bias=vec[:E].contiguous(), shared_gate=sg), nbytes=route_bytes)
+    add("moe_route, softmax with a correction and two outputs that are no experts (like)",
+        lambda: ops.moe_route(x, wr, top, None, 1.0, score="softmax", correction=vec, identity=2), nbytes=route_bytes)
+    gus = torch.randn(T, 2 * (E * fe + fs), device=dev)
+    dense, share = ops.moe_route(x, wr8, top, None, 1.0, score="softmax"), torch.rand(T, device=dev)
+    act_bytes = T * (top * 2 * fe * 4 + E * fe * 2)
+    add("moe_act, the shared expert behind the routed ones (new)",
+        lambda: ops.moe_act(gus, dense, E, fe, 7.0, 1.702, torch.bfloat16, shared=(fs, 7.0, share)), nbytes=act_bytes + T * fs * (2 * 4 + 2))
+    gu = gus[:, :2 * E * fe].contiguous()
+    add("moe_act (like)", lambda: ops.moe_act(gu, dense, E, fe, 7.0, 1.702, torch.bfloat16), nbytes=act_bytes)
+    print(json.dumps({"metric": "tokens/s of the Pukatar design beside Vugedra at equal sizes (bfloat16, random weights)",
+                      "design": "pukatar", "prompt_tokens": 2048, "decode_context": 1024, "steps": args.steps,
+                      "warmup": args.warmup, "sizes": sizes, "kernels_at_w4096": kernels,
+                      "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": round(tensor_peak / 1e12, 1), "source": pk["source"]},
+                      "l2": "kernel timings: a 256 MB buffer is overwritten between launches; steps read every weight"}))
+    return 0
+
+
 def komazen_bench(args, pk, measure) -> int:
     """`--design komazen`: the design beside Qwen3 (the closest model: softmax attention and a dense gated feed-forward
     in every layer) at equal width, heads, feed-forward, depth and vocabulary, and its kernels beside their like."""
@@ -1140,6 +1322,8 @@ def design_bench(args, pk) -> int:
         return komazen_bench(args, pk, measure)
     if args.design == "vugedra":
         return vugedra_bench(args, pk, measure)
+    if args.design == "pukatar":
+        return pukatar_bench(args, pk, measure)
     sizes = {}
     for name, (width, ff, heads, kv, layers) in DESIGN_SIZES.items():
         if args.sizes and name not in args.sizes.split(","):
@@ -1259,9 +1443,9 @@ def main() -> int:
     ap.add_argument("--points", default=",".join(ALL_POINTS),
                     help="which extra measurements to take: " + ",".join(ALL_POINTS))
     ap.add_argument("--no-points", action="store_true", help="the headline, prefill and e2e only")
-    ap.add_argument("--design", choices=["tobovik", "gubidra", "komazen", "vugedra"],
+    ap.add_argument("--design", choices=["tobovik", "gubidra", "komazen", "vugedra", "pukatar"],
                     help="instead of the default workload: this design beside its closest model (tobovik and komazen beside "
-                         "Qwen3, gubidra beside tobovik, vugedra beside gubidra) at equal sizes, and its kernels")
+                         "Qwen3, gubidra beside tobovik, vugedra beside gubidra, pukatar beside vugedra) at equal sizes, and its kernels")
     ap.add_argument("--sizes", default="", help="with --design: which of " + ",".join(DESIGN_SIZES) + " (default: all)")
     args = ap.parse_args()
 

@@ -32,6 +32,8 @@ class DeltaRuleMixer(BranchMixer):
     graph_safe = True            # kernels on the current stream only; their grids follow the step's entries
     any_division_safe = False
 
+    PADDED = (32, 64, 128, 256)  # what the kernels are instantiated for
+
     _DEFAULT_NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                       "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "b": "b_proj.weight",
                       "a1": "a_proj.0.weight", "a2": "a_proj.1.weight", "dt": "dt_bias", "A": "A_log", "g1": "g_proj.0.weight",
@@ -51,11 +53,10 @@ class DeltaRuleMixer(BranchMixer):
         self.channels = 2 * self.G * self.D + self.H * self.V    # what passes the convolutions
         self.out_width = self.H * self.V
         self.conv_w = self.w_decay = self.w_gate = self.dt_bias = self.a_log = self.norm_w = None
-        self.padded = self.D
-        if self.device.type == "cuda":
-            if not ops.delta_supported(self.D, self.V):
-                raise ValueError(f"the delta rule: a state of {self.D} x {self.V} per head is more than its kernels take")
-            self.padded = ops.delta_padded(self.D)
+        # rows of a head's state as the kernels keep them
+        self.padded = next((n for n in self.PADDED if self.D <= n), 0)
+        if not self.padded or (self.device.type == "cuda" and not ops.delta_supported(self.D, self.V)):
+            raise ValueError(f"the delta rule: a state of {self.D} x {self.V} per head is more than its kernels take")
 
     def parameters(self) -> Dict[str, ParamSpec]:
         n, W = self.names, self.hidden
