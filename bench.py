@@ -882,7 +882,7 @@ def pukatar_bench(args, pk, measure) -> int:
     run = lambda b, n, single: ops.delta_rule(proj[:n], (0, C, C + H, C + H + rank), (rank, rank), conv, lowa, lowa, dt, al, nw, 1e-5, 1.0, out[:n], 0,
                                               state, b, H, H, D, V, single=single)
     # flops of the recurrence itself: decay, two products with the state, the write (7 per entry of S)
-    add(f"delta rule, one portion of {T} tokens, {H} heads of {D} x {V}: convolutions, projections, recurrence, gated norm (new; 4 kernels)",
+    add(f"delta rule, one portion of {T} tokens, {H} heads of {D} x {V}: convolutions, projections, recurrence, gated norm (new; 5 kernels)",
         lambda: run(prompt, T, False), flops=7.0 * T * H * D * V, peak=fma_peak, peak_name="nominal_f32_fma_rate")
     q_g, st_g = torch.randn(T, 4 * H * D + rank, device=dev), torch.zeros(Bd, H, D, V, device=dev)
     w2t, b2 = torch.randn(rank, H * D, device=dev) * 0.1, torch.zeros(H * D, device=dev)

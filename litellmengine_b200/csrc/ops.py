@@ -1021,17 +1021,21 @@ def delta_rule(proj: torch.Tensor, offs, ranks, conv_w: torch.Tensor, w_decay: t
         _check(f(*args, _ptr(batch.entry_slot), _ptr(batch.entry_q_start), batch.num_entries, H, G, D, V, _stream()), "delta_step")
         return
     DP, VP = delta_padded(D), (V + 3) // 4 * 4
-    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
-    qn, kn, vn, kq, beta = new(T, G, DP), new(T, G, DP), new(T, H, VP), new(T, G), new(T, H)
-    decay = new(T, H, DP) if D == DP else torch.zeros((T, H, DP), dtype=torch.float32, device=dev)
-    gate, o = new(T, H, V), new(T, H, V)
+    chunks = T // 4 + batch.num_entries + 1                 # places for what the four tokens of a chunk share
+    sizes = (T * H * DP,) + 2 * (T * G * DP,) + (T * H * VP, T * H, T * H * V, T * H * V) + 2 * (T * H * DP,) + (chunks * H * DP, chunks * H * 24)
+    starts = [0]
+    for n in sizes:
+        starts.append(starts[-1] + (n + 3) // 4 * 4)
+    room = torch.empty(starts[-1], dtype=torch.float32, device=dev)
+    if D != DP:
+        room[:sizes[0]].zero_()                             # decays behind a head's key width must be finite
+    decay, qn, kn, vn, beta, gate, o, pk, pq, total, num = (room.data_ptr() + 4 * n for n in starts[:-1])
     f = _fn("delta_rule", "llm_delta_scan",
-            head + [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int] + [c_void_p] * 9)
+            head + [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int] + [c_void_p] * 12)
     _check(f(*args, _ptr(batch.token_entry), _ptr(batch.entry_slot), _ptr(batch.entry_q_start), _ptr(batch.entry_q_len), T,
-             batch.num_entries, H, G, D, V, _ptr(qn), _ptr(kn), _ptr(vn), _ptr(kq), _ptr(beta), _ptr(decay), _ptr(gate), _ptr(o),
-             _stream()), "delta_scan")
+             batch.num_entries, H, G, D, V, qn, kn, vn, beta, decay, gate, o, pk, pq, total, num, _stream()), "delta_scan")
     global launch_count
-    launch_count += 3                          # four kernels in one call
+    launch_count += 4                          # five kernels in one call
 
 
 # ---- several residual streams ----------------------------------------------------------------------------
