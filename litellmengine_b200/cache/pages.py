@@ -8,7 +8,7 @@ Vocabulary
   slot    the index a live request holds from admission to release; it picks the request's
           row in every block table and in every state tensor.
   group   the stages (entries of the model's run order) whose caches have the same needs
-          (kv heads, head size, window).  A group has its own page pool, its own block
+          (kv heads, head size, window or chunk).  A group has its own page pool, its own block
           table and one tensor `[stages, pages, 2, kv_heads, page_size, head_dim]`; a page
           id covers that page in all of the group's stages.
   table   table[slot][i] = physical page holding positions [i*P, (i+1)*P) of that request.
@@ -99,6 +99,7 @@ class PagedNeed:
     window: Optional[int] = None      # None: every earlier position stays; w: only the last w
     value_dim: Optional[int] = None
     keep_first: int = 0               # with a window: the first so many positions of a request stay all the same
+    chunk: Optional[int] = None       # instead of a window: only the chunk of so many positions that the next one lies in
 
     @property
     def key_width(self) -> int:
@@ -185,7 +186,7 @@ class CacheManager:
         self.num_pages = (max_total_tokens + page_size - 1) // page_size
         # A request can be longer than the pool only if every group forgets old positions.
         stage_needs = [_needs_of(n) for n in stage_needs]
-        keeps_all = any(isinstance(n, PagedNeed) and n.window is None for ns in stage_needs for n in ns)
+        keeps_all = any(isinstance(n, PagedNeed) and n.window is None and n.chunk is None for ns in stage_needs for n in ns)
         self.max_request_tokens = max_request_tokens or max_total_tokens
         if keeps_all:
             self.max_request_tokens = min(self.max_request_tokens, self.num_pages * page_size)
@@ -230,6 +231,10 @@ class CacheManager:
         for i, g in enumerate(self.groups):
             if g.need.window is not None and g.need.keep_first:
                 _check(self._lib.hc_cache_set_head(self._h, i, int(g.need.keep_first)))
+            if g.need.chunk is not None:
+                if g.need.window is not None:
+                    raise CacheError("a cache group forgets by a window or by chunks, not both")
+                _check(self._lib.hc_cache_set_chunk(self._h, i, int(g.need.chunk)))
             g._bind(self._lib, self._h, i, max_slots, max_pages_per_request)
         self.state: Dict[object, object] = {}     # stage index or name -> device tensor [max_slots, *shape]
         self._extra_state = dict(extra_state or {})
@@ -338,7 +343,7 @@ class CacheManager:
 
     def commit(self, slot: int, new_len: int) -> int:
         """The step that filled positions up to new_len has been issued: record the length and
-        give back pages that a window has passed.  Returns the number of pages given back."""
+        give back pages that a window or a chunk has passed.  Returns the number of pages given back."""
         given = ctypes.c_int()
         _check(self._lib.hc_cache_commit(self._h, int(slot), int(new_len), ctypes.byref(given)))
         return given.value

@@ -10,11 +10,12 @@ from .gubidra import GubidraConfig
 from .komazen import KomazenConfig
 from .vugedra import VugedraConfig
 from .pukatar import PukatarConfig
+from .purivik import PurivikConfig
 
 __all__ = [
     "ConfigError", "config_class_for", "config_from_dict", "load_config",
     "register_architecture", "registered_architectures", "save_config",
     "unregister_architecture", "BlockSpec", "FeedForwardSpec", "MixerSpec", "ModelPlan",
     "NormSpec", "PositionSpec", "StageSpec", "Qwen3Config", "TobovikConfig", "GubidraConfig", "KomazenConfig", "VugedraConfig",
-    "PukatarConfig", "RejoinSpec",
+    "PukatarConfig", "PurivikConfig", "RejoinSpec",
 ]

@@ -42,6 +42,9 @@ class PositionSpec:
     frequencies: with pair(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(pair(fast)), 0),
     hi = min(ceil(pair(slow)), rotary_dim - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency
     is f_i / factor * ramp_i + f_i * (1 - ramp_i); `params` magnitude multiplies cos and sin.
+    `params` wavelengths = (factor, low, high, original) stretches them by wavelength instead: with l = 2 pi / f_i, f_i
+    stays where l < original/high, is divided by factor where l > original/low, and between the two it is
+    (1 - s) * f_i / factor + s * f_i with s = (original/l - low) / (high - low).
     kind 'rope_half': the same tables for pairs (i, i + rotary_dim/2), for mixers whose kernels take either layout.
     `params` carries what other kinds need.
     """
@@ -57,7 +60,8 @@ class MixerSpec:
 
     kind 'attention': grouped-query causal attention over the paged cache.
     `window` = None attends to every earlier key; an integer w attends to the
-    last w keys (the query's own included).  `has_kv` = False makes a mixer that
+    last w keys (the query's own included).  `chunk` = c cuts the sequence into chunks of c positions, counted from its
+    start, and a query attends to the keys of its own chunk up to its own (at most one of the two).  `has_kv` = False makes a mixer that
     projects only queries and reads the keys and values another stage wrote (the
     stage that runs it must then name that stage in `cache_from`).  `params`
     carries what other kinds of mixer need.
@@ -123,17 +127,19 @@ class MixerSpec:
     log_distance_bias: bool = False
     keep_first: int = 0                    # with a window: the sequence's first so many keys stay visible to every later query
     softmax_sink: Optional[float] = None   # a score whose exponential joins the softmax's denominator and carries no value
+    chunk: Optional[int] = None            # instead of a window: attention within chunks of so many positions
     learned_sink: bool = False             # the same with a learned score per query head (tensor 'sink' [heads], not scaled)
 
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
     """The per-token part of a layer.  kind 'swiglu': down(act(gate(x)) * up(x)) with act = silu, or what
-    `params` activation names ('silu', 'gelu_tanh': 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))).
+    `params` activation names ('silu', 'gelu_tanh': 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); 'clamped_swish' with
+    `params` limit: down(g * sigmoid(1.702 g) * (u + 1)), the gate value g clamped from above, the up value u on both sides).
     kind 'moe': routed experts; `intermediate_size` is one expert's, `params`: experts, top, groups
     (count, keep) or None, route_scale, limit (the experts' clamp), expert_prefix (expert e's tensors are
     '<expert_prefix><e>.gate' and so on), score, correction, router_bias, identity, activation, shared, shared_activation,
-    shared_limit, shared_gate (see `RoutedExperts`).
+    shared_limit, shared_gate, normalize, weight_on_input (see `RoutedExperts`).
     `tensor_names`: pairs (the part's own name for a tensor, its name in the model's files)."""
     kind: str
     intermediate_size: int = 0
@@ -158,7 +164,8 @@ class BlockSpec:
     rows of h are kept per request, layer and sublayer).
     arrangement 'sandwich_norm': h += norm1b(mixer(norm1(h))); h += norm2b(ffn(norm2(h))): a norm in front of each
     sublayer and one on its output (`mixer_post_norm`, `feed_forward_post_norm`, named `mixer_post_norm_name` and
-    `feed_forward_post_norm_name`).
+    `feed_forward_post_norm_name`).  A sublayer's normed output may be multiplied on its way: by a learned factor per
+    channel (`layer_scale_names`, one tensor [hidden] per sublayer) and by the constant `branch_scale`.
     arrangement 'parallel_pre_norm': h += mixer(u) + ffn(u) with u = norm1(h): one norm that both sublayers read
     (`feed_forward_norm` None).
     `feed_forward` None: a layer that is its mixer only.
@@ -182,6 +189,8 @@ class BlockSpec:
     feed_forward_post_norm: Optional[NormSpec] = None
     mixer_post_norm_name: str = "post_mixer_layernorm"
     feed_forward_post_norm_name: str = "post_feed_forward_layernorm"
+    layer_scale_names: Optional[Tuple[str, str]] = None
+    branch_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -202,10 +211,12 @@ class StageSpec:
 @dataclass(frozen=True)
 class RejoinSpec:
     """What happens to the residual stream x in front of a stage with `starts_pass` = t: x <- W [x; x0] + step[t], x0 the
-    embedding output, W [hidden, 2 hidden] the tensor `in_name` (x first), step [passes, hidden] the tensor `step_name`."""
+    embedding output, W [hidden, 2 hidden] the tensor `in_name` (x first), step [passes, hidden] the tensor `step_name`.
+    kind 'add': x <- x + x0 in front of every pass but the first, without tensors."""
     passes: int
     in_name: str = "loop.in"
     step_name: str = "loop.step"
+    kind: str = "linear"
 
 
 @dataclass(frozen=True)
@@ -238,6 +249,8 @@ class ModelPlan:
             raise ValueError("a norm on the embedding excludes an added position, a scale and several streams")
         if self.rejoin is not None and (self.embedding_position is not None or self.streams):
             raise ValueError("a rejoin with the embedding excludes an added position and several streams")
+        if self.rejoin is not None and self.rejoin.kind not in ("linear", "add"):
+            raise ValueError(f"rejoin {self.rejoin.kind!r}: 'linear' or 'add'")
         if not self.order:
             raise ValueError("the run order is empty")
         for s, st in enumerate(self.order):

@@ -5,7 +5,7 @@
 // one mma tile (rows past the group size are zero and never stored).
 //
 // For the token in row r (request slot s, position p), kv head c, split i of n:
-//     keys j in [lo + i*len, lo + (i+1)*len) ∩ [lo, p],  lo = 0 or p - window + 1
+//     keys j in [lo + i*len, lo + (i+1)*len) ∩ [lo, p],  lo = the first key the query sees (`first_visible`)
 //     per query head h of the group: s_j = (q_h . k_j) * scale, running max m, sum l of
 //     exp(s_j - m), acc = sum exp(s_j - m) v_j      -- softmax state and accumulators in 32-bit
 // (the running-maximum form of src/ops/attention.cu:577-668, which walks the keys one by one
@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(AD_THREADS) paged_decode_attention_kernel(
     if (t < 0) return;                                              // a padding entry of the row list: no work
     const int pos = positions[t];
     const int32_t* table = block_table + static_cast<size_t>(entry_slot[token_entry[t]]) * table_stride;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = first_visible(pos, window);
     const int n_keys = pos - lo + 1;
     // BIAS, with a window and kept first keys: the LAST split walks the kept keys below the window, [0, min(keep_first,
     // lo)), and the others share the window; the merge kernel adds it like any other split.

@@ -103,7 +103,7 @@ __global__ void __launch_bounds__(AD_THREADS + 32) paged_decode_attention_tma_ke
     if (t < 0) return;                                              // a padding entry of the row list: no work
     const int pos = positions[t];
     const int32_t* table = block_table + static_cast<size_t>(entry_slot[token_entry[t]]) * table_stride;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = first_visible(pos, window);
     const int n_keys = pos - lo + 1;
     // BIAS, with a window and kept first keys: the LAST split walks the kept keys below the window, [0, min(keep_first,
     // lo)), and the others share the window; the merge kernel adds it like any other split.

@@ -3,7 +3,7 @@
 // bfloat16 path for sizes its tuned kernels do not take.
 //
 // For the query token t of the request in slot s at position p, head h (kv head h / group):
-//     keys j in [lo, p],  lo = 0 or p - window + 1 with a window
+//     keys j in [lo, p],  lo = the first key the query sees (0, a window's edge or the start of its chunk)
 //     s_j = (q . k_j) * scale;  softmax over j in 32-bit;  out = sum_j p_j v_j
 // with the running-maximum form of src/ops/attention.cu:204-249 applied to tiles of 32 keys
 // (the reference folds one key at a time; its paged kernel is src/ops/attention.cu:577-668).
@@ -81,7 +81,7 @@ __global__ void paged_attention_generic_kernel(
     const int pos = positions[t];
     const int slot = entry_slot[token_entry[t]];
     const int32_t* table = block_table + static_cast<size_t>(slot) * table_stride;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = first_visible(pos, window);
     const size_t khead = static_cast<size_t>(page_size) * d;        // one kv head inside a page of keys
     const size_t vrow = value_row_stride > 0 ? static_cast<size_t>(value_row_stride) : static_cast<size_t>(dv);
     const size_t vhead = static_cast<size_t>(page_size) * vrow;     // and inside a page of values

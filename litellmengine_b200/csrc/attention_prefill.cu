@@ -87,7 +87,7 @@ __global__ void __launch_bounds__(AP_THREADS) paged_prefill_attention_kernel(
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
     const int pos_first = past + q0, pos_last = past + q0 + rows_here - 1;
-    const int k_lo = (window > 0 && pos_first - window + 1 > 0) ? ((pos_first - window + 1) / AP_BN) * AP_BN : 0;
+    const int k_lo = first_visible(pos_first, window) / AP_BN * AP_BN;
     // EXT, with a window: the sequence's first `keep_first` keys stay visible.  The tiles that hold them and lie wholly
     // below the window's first tile are walked first; kept keys inside the window's tiles are a matter of the mask.
     const int keep = (EXT && window > 0) ? keep_first : 0;
@@ -149,8 +149,9 @@ __global__ void __launch_bounds__(AP_THREADS) paged_prefill_attention_kernel(
     float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.0f, l1 = 0.0f;      // rows lane/4 and lane/4 + 8
     const int r0 = warp * 16 + (lane >> 2);
     const int pos0 = past + q0 + r0, pos1 = pos0 + 8;
-    const int lo0 = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
-    const int lo1 = (window > 0 && pos1 - window + 1 > 0) ? pos1 - window + 1 : 0;
+    const int lo0 = first_visible(pos0, window);
+    const int lo1 = first_visible(pos1, window);
+    const int lo_last = first_visible(pos_last, window);
     const bool live0 = r0 < rows_here, live1 = r0 + 8 < rows_here;
     // a learned bias by distance, one row of [heads, distances] per head, already in the exp2 domain
     const float* bias_h = (EXT && dist_bias && dist_len > 0) ? dist_bias + static_cast<size_t>(h) * dist_len : nullptr;
@@ -212,7 +213,7 @@ __global__ void __launch_bounds__(AP_THREADS) paged_prefill_attention_kernel(
         ldmatrix_x4_trans(vf[0], v_addr(0));
         ldmatrix_x4_trans(vf[1], v_addr(1));
         // mask, scale into the exp2 domain, running max
-        const bool need_mask = (kt + AP_BN - 1 > pos_first) || (window > 0);
+        const bool need_mask = (kt + AP_BN - 1 > pos_first) || (kt < lo_last);        // lo_last: no row of the tile sees a key below its own edge
         float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
         for (int nb = 0; nb < AP_BN / 8; ++nb) {

@@ -171,7 +171,7 @@ __global__ void __launch_bounds__(64 + 128 * HEADS, 1) paged_prefill_attention_t
     const int32_t* table = block_table + static_cast<size_t>(entry_slot[e]) * table_stride;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int pos_first = past + q0, pos_last = past + q0 + rows_here - 1;
-    const int k_lo = (window > 0 && pos_first - window + 1 > 0) ? ((pos_first - window + 1) / T5_BN) * T5_BN : 0;
+    const int k_lo = first_visible(pos_first, window) / T5_BN * T5_BN;
     const int n_tiles = (pos_last - k_lo) / T5_BN + 1;
     const int total = 2 * n_tiles;                                // pass A then pass B over the same tiles
 
@@ -303,14 +303,14 @@ __global__ void __launch_bounds__(64 + 128 * HEADS, 1) paged_prefill_attention_t
         const int row = quarter * 32 + lane;
         const unsigned lane_addr = static_cast<unsigned>(quarter * 32) << 16;
         const int pos = (row < rows_here) ? past + q0 + row : -1;
-        const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+        const int lo = first_visible(pos, window), lo_last = first_visible(pos_last, window);
         float m = -CUDART_INF_F, l = 0.0f;
         bool ok = true;
         for (int u = 0; ok && u < n_tiles; ++u) {                 // pass A: maxima
             const int sb = u & 1, kt = k_lo + u * T5_BN;
             if (!t5_wait(&s_full[sb], (u >> 1) & 1, &abort_flag, status, row_base)) { ok = false; break; }
             t5_fence_after();
-            const bool full_tile = (kt + T5_BN - 1 <= pos_first) && (window <= 0) && (rows_here == T5_BM);
+            const bool full_tile = (kt + T5_BN - 1 <= pos_first) && (kt >= lo_last) && (rows_here == T5_BM);
             unsigned r[2][32];                                    // both halves of the row are requested at once
             t5_ld32(tmem + lane_addr + s_col(g, sb), r[0]);
             t5_ld32(tmem + lane_addr + s_col(g, sb) + 32, r[1]);
@@ -336,7 +336,7 @@ __global__ void __launch_bounds__(64 + 128 * HEADS, 1) paged_prefill_attention_t
             const int sb = u & 1, v = u - n_tiles, kt = k_lo + v * T5_BN;
             if (!t5_wait(&s_full[sb], (u >> 1) & 1, &abort_flag, status, row_base)) { ok = false; break; }
             t5_fence_after();
-            const bool full_tile = (kt + T5_BN - 1 <= pos_first) && (window <= 0) && (rows_here == T5_BM);
+            const bool full_tile = (kt + T5_BN - 1 <= pos_first) && (kt >= lo_last) && (rows_here == T5_BM);
             unsigned pk[32], r[2][32];
             t5_ld32(tmem + lane_addr + s_col(g, sb), r[0]);
             t5_ld32(tmem + lane_addr + s_col(g, sb) + 32, r[1]);
@@ -485,7 +485,7 @@ __global__ void __launch_bounds__(T5O_THREADS, 1) paged_prefill_attention_tcgen0
     const int32_t* table = block_table + static_cast<size_t>(entry_slot[e]) * table_stride;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int pos_first = past + q0, pos_last = past + q0 + rows_here - 1;
-    const int k_lo = (window > 0 && pos_first - window + 1 > 0) ? ((pos_first - window + 1) / T5O_BN) * T5O_BN : 0;
+    const int k_lo = first_visible(pos_first, window) / T5O_BN * T5O_BN;
     const int n_tiles = (pos_last - k_lo) / T5O_BN + 1;
 
     if (tid == 0) {
@@ -650,7 +650,7 @@ __global__ void __launch_bounds__(T5O_THREADS, 1) paged_prefill_attention_tcgen0
         const unsigned my_s = tmem + lane_addr + s_col(g) + half * 64;
         const unsigned my_o = tmem + lane_addr + o_col(g) + half * 64;
         const int pos = (row < rows_here) ? past + q0 + row : -1;
-        const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+        const int lo = first_visible(pos, window), lo_last = first_visible(pos_last, window);
         float m = -CUDART_INF_F, l = 0.0f;                        // m: the reference maximum, in units of log2
         bool ok = true;
         // with BIAS the scores are turned into their final form (units of log2) as they arrive, and `eff` is 1
@@ -686,7 +686,7 @@ __global__ void __launch_bounds__(T5O_THREADS, 1) paged_prefill_attention_tcgen0
             // number of times as the others, and touches nothing else.
             if (ok && !t5_wait(&s_full[g], j & 1, &abort_flag, status, row_base)) ok = false;
             t5_fence_after();
-            const bool full_tile = (kt + 63 <= pos_first) && (window <= 0) && (rows_here == T5_BM);
+            const bool full_tile = (kt + 63 <= pos_first) && (kt >= lo_last) && (rows_here == T5_BM);
             unsigned ra[32], rb[32];
             float mx = -CUDART_INF_F;
             if (ok) {

@@ -88,6 +88,21 @@ __device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
     *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
 }
 
+// A gated feed-forward's clamped middle: the gate, clamped from above, through g * sigmoid(alpha g), times the up value
+// clamped on both sides plus `shift`.  limit = infinity, alpha = 1, shift = 0 is silu(gate) * up.
+__device__ __forceinline__ float clamped_swish(float g, float u, float limit, float alpha, float shift) {
+    const float gc = fminf(g, limit), uc = fminf(fmaxf(u, -limit), limit);
+    return (gc / (1.0f + expf(-alpha * gc))) * (uc + shift);
+}
+#define CLAMPED_SWISH_ALPHA 1.702f
+
+// The first key that the query at `pos` sees.  span > 0: a sliding window, the last `span` keys, its own included.
+// span < 0: chunks of -span positions counted from the sequence's start, each query its own chunk's keys.  0: every key.
+__device__ __forceinline__ int first_visible(int pos, int span) {
+    if (span > 0) return max(pos - span + 1, 0);
+    return span < 0 ? pos - pos % -span : 0;
+}
+
 // ---- programmatic dependent launch -----------------------------------------------------------
 // Every kernel of the engine is launched with the "programmatic stream serialization" attribute
 // and begins with `pdl_begin()`: it lets the NEXT kernel in the stream be scheduled onto SMs

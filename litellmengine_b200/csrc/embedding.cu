@@ -4,6 +4,7 @@
 // with one element per thread and a blocking read of its error flag (src/layers/embedding.cu:91-158).
 // A negative id -1-j stands for feedback[j]: the token that the previous step sampled into a
 // device buffer, which the host has not read yet when it launches this step.
+// `keep` (optional) receives the same rows once more, for designs that come back to the embedding output later.
 //
 // Also here: the small scatter that applies a step's block-table changes on the device.
 #include "common.cuh"
@@ -12,15 +13,19 @@ template <typename T>
 __global__ void embedding_gather_kernel(const int32_t* __restrict__ ids, const T* __restrict__ table,
                                         float* __restrict__ out, int hidden, int vocab,
                                         int32_t* __restrict__ status, const int32_t* __restrict__ feedback,
-                                        int feedback_len, float scale) {
+                                        int feedback_len, float scale, float* __restrict__ keep) {
     pdl_begin();
     const int t = blockIdx.x;
     int id = ids[t];
     if (id < 0 && feedback != nullptr && -1 - id < feedback_len) id = feedback[-1 - id];
     float* o = out + static_cast<size_t>(t) * hidden;
+    float* o2 = keep ? keep + static_cast<size_t>(t) * hidden : nullptr;      // the same row once more
     if (id < 0 || id >= vocab) {
         if (threadIdx.x == 0 && atomicCAS(status, 0, 1) == 0) status[1] = t;
-        for (int h = threadIdx.x; h < hidden; h += blockDim.x) o[h] = 0.0f;
+        for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+            o[h] = 0.0f;
+            if (o2) o2[h] = 0.0f;
+        }
         return;
     }
     const T* row = table + static_cast<size_t>(id) * hidden;
@@ -31,26 +36,32 @@ __global__ void embedding_gather_kernel(const int32_t* __restrict__ ids, const T
 #pragma unroll
             for (int i = 0; i < 8; ++i) v[i] *= scale;      // a design's embedding scale, applied in 32-bit (1: exact)
             store8(o + h, v);
+            if (o2) store8(o2 + h, v);
         }
     } else {
-        for (int h = threadIdx.x; h < hidden; h += blockDim.x) o[h] = to_f32(row[h]) * scale;
+        for (int h = threadIdx.x; h < hidden; h += blockDim.x) {
+            const float v = to_f32(row[h]) * scale;
+            o[h] = v;
+            if (o2) o2[h] = v;
+        }
     }
 }
 
 extern "C" int llm_embedding_gather(const int32_t* ids, const void* table, int table_dtype, float* out,
                                     int num_tokens, int hidden, int vocab, int32_t* status,
-                                    const int32_t* feedback, int feedback_len, float scale, uintptr_t stream) {
+                                    const int32_t* feedback, int feedback_len, float scale, float* keep,
+                                    uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
     if (hidden <= 0 || vocab <= 0) return LLM_REFUSED_SIZE;
-    if ((hidden & 7) == 0 && (!aligned16(table) || !aligned16(out))) return LLM_REFUSED_ALIGN;
+    if ((hidden & 7) == 0 && (!aligned16(table) || !aligned16(out) || (keep && !aligned16(keep)))) return LLM_REFUSED_ALIGN;
     const int threads = hidden >= 2048 ? 256 : 128;
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
     if (table_dtype == LLM_DT_F32)
         launch_pdl((embedding_gather_kernel<float>), dim3(num_tokens), dim3(threads), 0, s, 
-            ids, static_cast<const float*>(table), out, hidden, vocab, status, feedback, feedback_len, scale);
+            ids, static_cast<const float*>(table), out, hidden, vocab, status, feedback, feedback_len, scale, keep);
     else if (table_dtype == LLM_DT_BF16)
         launch_pdl((embedding_gather_kernel<bf16>), dim3(num_tokens), dim3(threads), 0, s, 
-            ids, static_cast<const bf16*>(table), out, hidden, vocab, status, feedback, feedback_len, scale);
+            ids, static_cast<const bf16*>(table), out, hidden, vocab, status, feedback, feedback_len, scale, keep);
     else
         return LLM_REFUSED_DTYPE;
     return launch_status();

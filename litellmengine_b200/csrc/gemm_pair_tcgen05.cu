@@ -171,13 +171,14 @@ __device__ __forceinline__ bool gp_unit(const GpPlan& p, int i, int cluster, int
 // MODE 0: y[T, N] = x . w^T.  MODE 1: w is [gate; up] of 2 * inter rows, y[T, inter] = silu(gate) * up.
 // MODE 2: y[T, N] (float32) += x . w^T: the product joins the residual stream where it lies.
 // MODE 3: MODE 1 with the tanh form of gelu in place of silu (an instantiation of its own).
+// MODE 4: the clamped form with `limit` (`clamped_swish`, alpha 1.702, up value plus one).
 // w_map, w_map2: the same weights read in boxes of 128 and 64 rows (for whole tiles and for halves).
-#define GP_GATED(MODE) ((MODE) == 1 || (MODE) == 3)
+#define GP_GATED(MODE) ((MODE) == 1 || (MODE) >= 3)
 template <int MODE, typename TO>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GP_THREADS, 1) linear_pair_tcgen05_kernel(
     const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map,
     const __grid_constant__ CUtensorMap w_map2, TO* __restrict__ y,
-    int T, int N, int K, int inter, GpPlan plan, int32_t* __restrict__ status) {
+    int T, int N, int K, int inter, GpPlan plan, int32_t* __restrict__ status, float limit) {
     pdl_invite();
     constexpr int TILE_ELEMS = GP_BM * GP_BK;
     extern __shared__ unsigned char smem_dyn[];
@@ -302,7 +303,8 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GP_THREADS, 1) linea
                     for (int e = 0; e < 32; ++e) {
                         const float gate = __bfloat162float(__float2bfloat16_rn(__uint_as_float(g[e])));
                         const float upv = __bfloat162float(__float2bfloat16_rn(__uint_as_float(up[e])));
-                        v[e] = (MODE == 3 ? gp_gelu_tanh(gate) : gp_silu(gate)) * upv;
+                        if (MODE == 4) v[e] = clamped_swish(gate, upv, limit, CLAMPED_SWISH_ALPHA, 1.0f);
+                        else v[e] = (MODE == 3 ? gp_gelu_tanh(gate) : gp_silu(gate)) * upv;
                     }
                 } else {
                     unsigned r[32];
@@ -427,7 +429,7 @@ extern "C" int llm_linear_pair_efficiency(int T, int N, int K, int gate_up) {
 
 template <int MODE, typename TO>
 static int gp_launch(const bf16* x, const bf16* w, void* y, int T, int N, int K, int inter, long long w_rows, int32_t* status,
-                     cudaStream_t s) {
+                     cudaStream_t s, float limit = 0.0f) {
     CUtensorMap x_map, w_map, w_map2;
     if (!gp_encode(&x_map, x, T, K, GP_BM) || !gp_encode(&w_map, w, w_rows, K, GP_BN / 2) ||
         !gp_encode(&w_map2, w, w_rows, K, GP_BN / 4))
@@ -443,7 +445,7 @@ static int gp_launch(const bf16* x, const bf16* w, void* y, int T, int N, int K,
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     launch_pdl(kern, dim3(2 * clusters), dim3(GP_THREADS), smem, s, x_map, w_map, w_map2, static_cast<TO*>(y), T, N, K,
-               inter, plan, status);
+               inter, plan, status, limit);
     return launch_status();
 }
 
@@ -467,12 +469,15 @@ extern "C" int llm_linear_pair(const void* x, const void* w, void* y, int out_dt
 }
 
 // x: bfloat16 [T, K]; w: bfloat16 [2 * inter, K] = [gate; up]; y: bfloat16 [T, inter] = silu(gate) * up, gate and up
-// rounded to bfloat16 first.
-extern "C" int llm_linear_pair_silu_mul(const void* x, const void* w, void* y, int T, int inter, int K, int act,
+// rounded to bfloat16 first.  act 1: the tanh form of gelu instead of silu; 2: the clamped form with `limit`.
+extern "C" int llm_linear_pair_silu_mul(const void* x, const void* w, void* y, int T, int inter, int K, int act, float limit,
                                         int32_t* status, uintptr_t stream) {
-    if (!llm_linear_pair_supported(T, inter, K) || act < 0 || act > 1) return LLM_REFUSED_SIZE;
+    if (!llm_linear_pair_supported(T, inter, K) || act < 0 || act > 2 || (act == 2 && !(limit > 0.0f))) return LLM_REFUSED_SIZE;
     if (!aligned16(x) || !aligned16(w) || !aligned16(y) || status == nullptr) return LLM_REFUSED_ALIGN;
     if (!gp_ready()) return LLM_REFUSED_SIZE;
+    if (act == 2)
+        return gp_launch<4, bf16>(static_cast<const bf16*>(x), static_cast<const bf16*>(w), y, T, inter, K, inter, 2LL * inter,
+                                  status, reinterpret_cast<cudaStream_t>(stream), limit);
     if (act == 1)               // the tanh form of gelu
         return gp_launch<3, bf16>(static_cast<const bf16*>(x), static_cast<const bf16*>(w), y, T, inter, K, inter, 2LL * inter,
                                   status, reinterpret_cast<cudaStream_t>(stream));

@@ -75,6 +75,7 @@ struct Pool {
 
 struct Group {
     int page_size, window, max_pages;                    // window < 0: every earlier position stays
+    int chunk = 0;                                       // > 0, instead of a window: only the chunk of the next position stays
     int head = 0;                                        // with a window: the first `head` positions stay all the same
     Pool pool;
     std::vector<int32_t> table;                          // [slots][max_pages], -1 where nothing is held
@@ -103,11 +104,11 @@ struct Group {
         return HC_OK;
     }
     // Pages every position of which lies before the window of the next query (position `length`,
-    // which sees keys > length - window) go back.  Returns how many through `given`.
+    // which sees keys > length - window, or those of its own chunk) go back.  Returns how many through `given`.
     int trim_window(int slot, long long length, int* given) {
         *given = 0;
-        if (window < 0) return HC_OK;
-        const long long first_needed = std::max(0LL, length - window + 1);
+        if (window < 0 && chunk <= 0) return HC_OK;
+        const long long first_needed = chunk > 0 ? length / chunk * chunk : std::max(0LL, length - window + 1);
         const int keep_from = static_cast<int>(std::min<long long>(first_needed / page_size, num_logical[slot]));
         const int lo = std::max<int>(first_held[slot], pages_for(head));     // the head's pages never go back here
         if (keep_from <= lo) return HC_OK;
@@ -265,6 +266,14 @@ int hc_cache_set_head(void* c, int g, int head) {
     Cache* cc = cache_of(c);
     if (g < 0 || g >= static_cast<int>(cc->groups.size()) || head < 0) return fail(HC_MISUSE, "no such group, or a negative head");
     cc->groups[g].head = head;
+    return HC_OK;
+}
+// Group g keeps, of every request, the chunk of `chunk` positions (counted from 0) that its next position lies in.
+int hc_cache_set_chunk(void* c, int g, int chunk) {
+    Cache* cc = cache_of(c);
+    if (g < 0 || g >= static_cast<int>(cc->groups.size()) || chunk <= 0 || cc->groups[g].window >= 0)
+        return fail(HC_MISUSE, "no such group, a chunk that is not positive, or a group with a window");
+    cc->groups[g].chunk = chunk;
     return HC_OK;
 }
 void hc_cache_delete(void* c) { delete cache_of(c); }

@@ -17,6 +17,7 @@
 //                    `bias` (float32 [router outputs], optional) joins the logits themselves, before any score.
 //                    `shared_w` (float32 [W], optional): one more row, whose product's sigmoid goes to `share` [tokens]
 //                    (the weight of an expert that every token runs).
+//                    `normalize` 0: the weights are the chosen scores themselves times route_scale, not divided by their sum.
 //                    The experts' activation: g = min(gate, limit), u = clamp(up, -limit, limit),
 //                    w * g * sigmoid(alpha g) * (u + up_shift); limit = infinity, alpha = 1, up_shift = 0 is
 //                    the plain silu(gate) * up.
@@ -36,7 +37,8 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
                                  int32_t* __restrict__ ids, float* __restrict__ weights, int num_tokens, int W, int E,
                                  int top, int groups, int keep, float route_scale, int vec, int softmax,
                                  const float* __restrict__ correction, int identity, float* __restrict__ idw,
-                                 const float* __restrict__ bias, const float* __restrict__ shared_w, float* __restrict__ share) {
+                                 const float* __restrict__ bias, const float* __restrict__ shared_w, float* __restrict__ share,
+                                 int normalize) {
     pdl_begin();
     extern __shared__ float smem[];
     const int G = groups > 0 ? groups : 1;
@@ -154,7 +156,7 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
                 total += sc[best];
             }
         }
-        const float inv = route_scale / (total + 1e-20f);
+        const float inv = normalize ? route_scale / (total + 1e-20f) : route_scale;
         float own = 0.0f;                            // what the token gets of its own input
         for (int n = 0; n < top; ++n) {
             const int e = chosen[n];
@@ -174,7 +176,7 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
 extern "C" int llm_moe_route(const void* x, int x_dtype, const float* wr, float* dense, int32_t* ids, float* weights,
                              int num_tokens, int W, int E, int top, int groups, int keep, float route_scale,
                              int softmax, const float* correction, int identity, float* idw, const float* bias,
-                             const float* shared_w, float* share, uintptr_t stream) {
+                             const float* shared_w, float* share, int normalize, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
     if (identity < 0 || identity >= E || (identity > 0 && !idw)) return LLM_REFUSED_SIZE;
     if (W <= 0 || E <= 0 || top <= 0 || top > E || top > 64 || groups < 0) return LLM_REFUSED_SIZE;
@@ -195,7 +197,7 @@ extern "C" int llm_moe_route(const void* x, int x_dtype, const float* wr, float*
         }                                                                                                           \
         launch_pdl(kern, grid, dim3(MOE_ROUTE_THREADS), smem, s, static_cast<const TX*>(x), wr, dense, ids, weights,  \
                    num_tokens, W, E, top, groups, keep, route_scale, vec, softmax, correction, identity, idw, bias, \
-                   shared_w, share);                                                                                \
+                   shared_w, share, normalize);                                                                     \
     } while (0)
     if (x_dtype == LLM_DT_F32) LAUNCH(float);
     else if (x_dtype == LLM_DT_BF16) LAUNCH(bf16);
@@ -204,10 +206,11 @@ extern "C" int llm_moe_route(const void* x, int x_dtype, const float* wr, float*
     return launch_status();
 }
 
-// An expert's activation: the clamped gate through g * sigmoid(alpha g), times the clamped up value plus `shift`.
-__device__ __forceinline__ float moe_activate(float g, float u, float limit, float alpha, float shift) {
-    const float gc = fminf(g, limit), uc = fminf(fmaxf(u, -limit), limit);
-    return (gc / (1.0f + expf(-alpha * gc))) * (uc + shift);
+// An expert's weighted activation.  `on_input`: the expert runs on w * x instead of x, which scales its gate and up values
+// (they are linear in x) and leaves its output as it is; else its output is multiplied by w.
+__device__ __forceinline__ float moe_activate(float g, float u, float w, int on_input, float limit, float alpha, float shift) {
+    if (on_input) return clamped_swish(w * g, w * u, limit, alpha, shift);
+    return w * clamped_swish(g, u, limit, alpha, shift);
 }
 __device__ __forceinline__ void moe_store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
 __device__ __forceinline__ void moe_store4(bf16* p, const float (&v)[4]) {
@@ -226,7 +229,7 @@ __device__ __forceinline__ void moe_store4(bf16* p, const float (&v)[4]) {
 template <typename TO, int VEC>
 __global__ void moe_act_kernel(const float* __restrict__ gu, int parts, long long part_stride,
                                const float* __restrict__ dense, TO* __restrict__ act, int E, int ff_routed, float limit,
-                               float alpha, float shift, int ffs, float limit_s, const float* __restrict__ share) {
+                               float alpha, float shift, int ffs, float limit_s, const float* __restrict__ share, int on_input) {
     pdl_begin();
     const int slots = E + (ffs > 0 ? 1 : 0);
     const long long t = blockIdx.x / slots;
@@ -254,7 +257,7 @@ __global__ void moe_act_kernel(const float* __restrict__ gu, int parts, long lon
             }
         }
 #pragma unroll
-        for (int c = 0; c < VEC; ++c) out[c] = w * moe_activate(g[c], u[c], limit, alpha, shift);
+        for (int c = 0; c < VEC; ++c) out[c] = moe_activate(g[c], u[c], w, routed ? on_input : 0, limit, alpha, shift);
     }
     TO* o = act + t * width + first + f;
     if (VEC == 4) moe_store4(o, out);
@@ -263,7 +266,7 @@ __global__ void moe_act_kernel(const float* __restrict__ gu, int parts, long lon
 
 extern "C" int llm_moe_act(const float* gu, int parts, long long part_stride, const float* dense, void* act,
                            int act_dtype, int num_tokens, int E, int ff, float limit, float alpha, float shift,
-                           int ffs, float limit_s, const float* share, uintptr_t stream) {
+                           int ffs, float limit_s, const float* share, int on_input, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
     // E = 0: a shared expert alone
     if (E < 0 || ff < 0 || ffs < 0 || (E > 0 && (ff <= 0 || !(limit > 0.0f) || !dense)) || (ffs > 0 && !(limit_s > 0.0f)) || E + ffs <= 0)
@@ -278,7 +281,7 @@ extern "C" int llm_moe_act(const float* gu, int parts, long long part_stride, co
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define LAUNCH(TO, V)                                                                                          \
     launch_pdl((moe_act_kernel<TO, V>), grid, dim3(128), 0, s, gu, parts, part_stride, dense, static_cast<TO*>(act), E, ff, \
-               limit, alpha, shift, ffs, limit_s, share)
+               limit, alpha, shift, ffs, limit_s, share, on_input)
     if (act_dtype == LLM_DT_F32) { if (vec) LAUNCH(float, 4); else LAUNCH(float, 1); }
     else if (act_dtype == LLM_DT_BF16) { if (vec) LAUNCH(bf16, 4); else LAUNCH(bf16, 1); }
     else return LLM_REFUSED_DTYPE;
@@ -364,7 +367,7 @@ template <typename TX, typename TW, typename TO>
 __global__ void moe_gate_up_sparse_kernel(const TX* __restrict__ x, const TW* __restrict__ wgu,
                                           const int32_t* __restrict__ ids, const float* __restrict__ weights,
                                           TO* __restrict__ act, int W, int ff, int top, float limit, float alpha, int vec,
-                                          float shift) {
+                                          float shift, int on_input) {
     pdl_begin();
     extern __shared__ __align__(16) float xs[];        // [W]
     const int pair = blockIdx.x, t = pair / top;
@@ -380,7 +383,7 @@ __global__ void moe_gate_up_sparse_kernel(const TX* __restrict__ x, const TW* __
             const TW* gr = wgu + (static_cast<size_t>(e) * 2 * ff + f) * W;
             float g, u;
             moe_dot2(gr, gr + static_cast<size_t>(ff) * W, xs, W, lane, vec, g, u);
-            out = wt * moe_activate(g, u, limit, alpha, shift);
+            out = moe_activate(g, u, wt, on_input, limit, alpha, shift);
         }
         if (lane == 0) act[static_cast<size_t>(pair) * ff + f] = from_f32<TO>(out);
     }
@@ -410,7 +413,7 @@ __global__ void moe_down_sparse_kernel(const TA* __restrict__ act, const TW* __r
 
 extern "C" int llm_moe_sparse(const void* x, int x_dtype, const void* wgu, const void* wd, int w_dtype, const int32_t* ids,
                               const float* weights, void* act, float* out, int num_tokens, int W, int ff, int E, int top,
-                              float limit, float alpha, float shift, long long down_stride, uintptr_t stream) {
+                              float limit, float alpha, float shift, long long down_stride, int on_input, uintptr_t stream) {
     if (num_tokens <= 0) return LLM_OK;
     if (W <= 0 || ff <= 0 || E <= 0 || top <= 0 || !(limit > 0.0f) || down_stride < static_cast<long long>(E) * ff) return LLM_REFUSED_SIZE;
     const size_t smem_a = static_cast<size_t>(W) * sizeof(float), smem_b = static_cast<size_t>(top) * ff * sizeof(float);
@@ -423,12 +426,12 @@ extern "C" int llm_moe_sparse(const void* x, int x_dtype, const void* wgu, const
     const dim3 block(MOE_SPARSE_WARPS * 32);
     if (x_dtype == LLM_DT_F32) {
         launch_pdl((moe_gate_up_sparse_kernel<float, float, float>), grid_a, block, smem_a, s, static_cast<const float*>(x),
-                   static_cast<const float*>(wgu), ids, weights, static_cast<float*>(act), W, ff, top, limit, alpha, vec, shift);
+                   static_cast<const float*>(wgu), ids, weights, static_cast<float*>(act), W, ff, top, limit, alpha, vec, shift, on_input);
         launch_pdl((moe_down_sparse_kernel<float, float>), grid_b, block, smem_b, s, static_cast<const float*>(act),
                    static_cast<const float*>(wd), ids, out, W, ff, top, down_stride, vec);
     } else if (x_dtype == LLM_DT_BF16) {
         launch_pdl((moe_gate_up_sparse_kernel<bf16, bf16, bf16>), grid_a, block, smem_a, s, static_cast<const bf16*>(x),
-                   static_cast<const bf16*>(wgu), ids, weights, static_cast<bf16*>(act), W, ff, top, limit, alpha, vec, shift);
+                   static_cast<const bf16*>(wgu), ids, weights, static_cast<bf16*>(act), W, ff, top, limit, alpha, vec, shift, on_input);
         launch_pdl((moe_down_sparse_kernel<bf16, bf16>), grid_b, block, smem_b, s, static_cast<const bf16*>(act),
                    static_cast<const bf16*>(wd), ids, out, W, ff, top, down_stride, vec);
     } else {
@@ -499,7 +502,7 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, const int32_t* __rest
 template <typename T>
 __global__ void moe_act_pairs_kernel(const T* __restrict__ gu, const int32_t* __restrict__ row_pair,
                                      const float* __restrict__ weights, T* __restrict__ act, int ff, float limit,
-                                     float alpha, int vec, float shift) {
+                                     float alpha, int vec, float shift, int on_input) {
     pdl_begin();
     const long long r = blockIdx.x;
     const float w = weights[row_pair[r]];
@@ -511,12 +514,12 @@ __global__ void moe_act_pairs_kernel(const T* __restrict__ gu, const int32_t* __
             load8(g + f, a);
             load8(g + ff + f, b);
 #pragma unroll
-            for (int c = 0; c < 8; ++c) a[c] = w * moe_activate(a[c], b[c], limit, alpha, shift);
+            for (int c = 0; c < 8; ++c) a[c] = moe_activate(a[c], b[c], w, on_input, limit, alpha, shift);
             store8(o + f, a);
         }
     } else {
         for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < ff; f += gridDim.y * blockDim.x) {
-            o[f] = from_f32<T>(w * moe_activate(to_f32(g[f]), to_f32(g[ff + f]), limit, alpha, shift));
+            o[f] = from_f32<T>(moe_activate(to_f32(g[f]), to_f32(g[ff + f]), w, on_input, limit, alpha, shift));
         }
     }
 }
@@ -565,7 +568,7 @@ extern "C" int llm_moe_sort(const int32_t* ids, int pairs, int E, int32_t* offs,
 // 2: combine (a = y [pairs, n], out = float32 [T, n], index = pos, `weights` an optional float32
 // [T, n] the sums start from, aligned like `out`).  n is the row width of `out`.
 extern "C" int llm_moe_rows(int which, const void* a, int dtype, const int32_t* index, const float* weights, void* out,
-                            int rows, int n, int top, float limit, float alpha, float shift, uintptr_t stream) {
+                            int rows, int n, int top, float limit, float alpha, float shift, int on_input, uintptr_t stream) {
     if (rows <= 0) return LLM_OK;
     if (n <= 0 || top <= 0 || which < 0 || which > 2) return LLM_REFUSED_SIZE;
     const int esz = dtype == LLM_DT_F32 ? 4 : 2;
@@ -581,9 +584,9 @@ extern "C" int llm_moe_rows(int which, const void* a, int dtype, const int32_t* 
         else return LLM_REFUSED_DTYPE;
     } else if (which == 1) {
         if (dtype == LLM_DT_F32) launch_pdl((moe_act_pairs_kernel<float>), grid, block, 0, s, static_cast<const float*>(a), index,
-                                            weights, static_cast<float*>(out), n, limit, alpha, vec, shift);
+                                            weights, static_cast<float*>(out), n, limit, alpha, vec, shift, on_input);
         else if (dtype == LLM_DT_BF16) launch_pdl((moe_act_pairs_kernel<bf16>), grid, block, 0, s, static_cast<const bf16*>(a),
-                                                  index, weights, static_cast<bf16*>(out), n, limit, alpha, vec, shift);
+                                                  index, weights, static_cast<bf16*>(out), n, limit, alpha, vec, shift, on_input);
         else return LLM_REFUSED_DTYPE;
     } else {
         if (dtype == LLM_DT_F32) launch_pdl((moe_combine_kernel<float>), grid, block, 0, s, static_cast<const float*>(a), index,

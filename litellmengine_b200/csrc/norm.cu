@@ -223,3 +223,142 @@ extern "C" int llm_rmsnorm_add(float* h, const void* y, int y_dtype, long long y
 #undef LAUNCH
     return launch_status();
 }
+
+// The step between two sublayers of a design that norms a sublayer's input AND its output, in 32-bit throughout:
+//     v      = h[row] + n(y[row]) * w_post (+ join[row])        n(a) = a * rsqrt(mean(a^2) + eps)
+//     h[row] = v                                                (with write_h; the stream is float32)
+//     out    = n(v) * w_pre                                     stored in the compute dtype
+// Without w_post, y joins as it is; y may be absent; y may come as the `parts` k-splits of a product, `part_stride`
+// elements apart, added in order as they are read.  `join` (optional, float32 like h) is one more summand: what a
+// design adds to the stream in front of a sublayer.  `w_post` carries whatever constant factors the sum has per
+// channel.  `rows` (optional) picks which rows are read, so a model's final norm runs only where logits are wanted
+// (h is then left alone).
+// One block per row.  REG: the row fits the block with eight neighbouring elements a thread (blockDim * 8 >= hidden),
+// which stay in registers between the two reductions, and everything the row needs is asked for before the first of
+// them.  Otherwise the row passes through shared memory.
+template <typename TY, typename TO, bool REG>
+__global__ void __launch_bounds__(1024) rmsnorm_sandwich_kernel(float* __restrict__ h, const TY* __restrict__ y, long long y_stride, int parts,
+                                        long long part_stride, const float* __restrict__ w_post, float eps_post,
+                                        const float* __restrict__ join, const float* __restrict__ w_pre, float eps_pre,
+                                        TO* __restrict__ out, const int32_t* __restrict__ rows, int hidden, int write_h) {
+    __shared__ float scratch[33];
+    if constexpr (REG) {
+        const int i = threadIdx.x * 8;
+        const bool mine = i < hidden;
+        float wp[8], wn[8];                             // the weights are the model's: read before the wait
+        if (mine && w_post) load8(w_post + i, wp);
+        if (mine) load8(w_pre + i, wn);
+        pdl_begin();
+        const size_t src = rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
+        float* hr = h + src * hidden;
+        float v[8] = {0, 0, 0, 0, 0, 0, 0, 0}, a[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+        if (mine) {
+            load8(hr + i, v);
+            if (join) {
+                float b[8];
+                load8(join + src * hidden + i, b);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) v[u] += b[u];
+            }
+            if (y) {
+                const TY* yr = y + src * y_stride + i;
+                load8(yr, a);
+#pragma unroll 4
+                for (int part = 1; part < parts; ++part) {
+                    float b[8];
+                    load8(yr + part * part_stride, b);
+#pragma unroll
+                    for (int u = 0; u < 8; ++u) a[u] += b[u];
+                }
+            }
+        }
+        if (y) {
+            float inv = 1.0f;
+            if (w_post) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int u = 0; u < 8; ++u) ss += a[u] * a[u];
+                inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_post);
+            }
+#pragma unroll
+            for (int u = 0; u < 8; ++u) v[u] += w_post ? (mine ? a[u] * inv * wp[u] : 0.0f) : a[u];
+        }
+        if (write_h && mine) store8(hr + i, v);
+        float ss = 0.0f;
+#pragma unroll
+        for (int u = 0; u < 8; ++u) ss += v[u] * v[u];
+        const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_pre);
+        if (mine) {
+#pragma unroll
+            for (int u = 0; u < 8; ++u) v[u] = v[u] * inv * wn[u];
+            store8(out + static_cast<size_t>(blockIdx.x) * hidden + i, v);
+        }
+    } else {
+        pdl_begin();
+        extern __shared__ __align__(16) float row_s[];
+        const size_t src = rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
+        float* hr = h + src * hidden;
+        const float* jr = join ? join + src * hidden : nullptr;
+        const TY* yr = y ? y + src * y_stride : nullptr;
+        float inv = 1.0f;
+        if (yr) {
+            float ss = 0.0f;
+            for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+                float a = to_f32(yr[i]);
+                for (int part = 1; part < parts; ++part) a += to_f32(yr[part * part_stride + i]);
+                row_s[i] = a;
+                ss += a * a;
+            }
+            if (w_post) inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_post);
+        }
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) {       // each thread meets the elements it wrote itself
+            float v = hr[i];
+            if (jr) v += jr[i];
+            if (yr) v += w_post ? row_s[i] * inv * w_post[i] : row_s[i];
+            row_s[i] = v;
+            if (write_h) hr[i] = v;
+            ss += v * v;
+        }
+        inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_pre);
+        TO* orow = out + static_cast<size_t>(blockIdx.x) * hidden;
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) orow[i] = from_f32<TO>(row_s[i] * inv * w_pre[i]);
+    }
+}
+
+// h: float32 [*, hidden]; y: [*, hidden] with `y_stride` elements a row, or null; w_post: float32 [hidden] or null; join:
+// float32 like h, or null; w_pre: float32 [hidden]; out: [num_rows, hidden]; rows: int32 [num_rows] or null.
+extern "C" int llm_rmsnorm_sandwich(float* h, const void* y, int y_dtype, long long y_stride, int parts, long long part_stride,
+                                    const float* w_post, float eps_post, const float* join, const float* w_pre, float eps_pre,
+                                    void* out, int out_dtype, const int32_t* rows, int num_rows, int hidden,
+                                    uintptr_t stream) {
+    if (num_rows <= 0) return LLM_OK;
+    if (hidden <= 0 || parts < 1 || (y && y_stride < hidden) || !w_pre || !out) return LLM_REFUSED_SIZE;
+    const size_t smem = static_cast<size_t>(hidden) * sizeof(float);
+    if (smem > 200 * 1024) return LLM_REFUSED_SIZE;
+    if (!y) y_dtype = LLM_DT_F32;
+    const int write_h = (y || join) && !rows;
+    const bool reg = hidden % 8 == 0 && hidden <= 8192 && aligned16(h) && aligned16(out) && aligned16(w_pre) &&
+                     (!y || (aligned16(y) && y_stride % 8 == 0 && part_stride % 8 == 0)) && (!w_post || aligned16(w_post)) &&
+                     (!join || aligned16(join));
+    const int threads = reg ? (hidden / 8 + 31) / 32 * 32 : (hidden >= 4096 ? 512 : (hidden >= 1024 ? 256 : 128));
+    cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define LAUNCH(TY, TO)                                                                                                   \
+    do {                                                                                                                 \
+        auto kern = reg ? rmsnorm_sandwich_kernel<TY, TO, true> : rmsnorm_sandwich_kernel<TY, TO, false>;                \
+        if (!reg && smem > 48 * 1024) {                                                                                  \
+            const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,                \
+                                                       static_cast<int>(smem));                                          \
+            if (e != cudaSuccess) return static_cast<int>(e);                                                            \
+        }                                                                                                                \
+        launch_pdl(kern, dim3(num_rows), dim3(threads), reg ? 0 : smem, s, h, static_cast<const TY*>(y), y_stride, parts, \
+                   part_stride, w_post, eps_post, join, w_pre, eps_pre, static_cast<TO*>(out), rows, hidden, write_h);   \
+    } while (0)
+    if (y_dtype == LLM_DT_F32 && out_dtype == LLM_DT_F32) LAUNCH(float, float);
+    else if (y_dtype == LLM_DT_F32 && out_dtype == LLM_DT_BF16) LAUNCH(float, bf16);
+    else if (y_dtype == LLM_DT_BF16 && out_dtype == LLM_DT_F32) LAUNCH(bf16, float);
+    else if (y_dtype == LLM_DT_BF16 && out_dtype == LLM_DT_BF16) LAUNCH(bf16, bf16);
+    else return LLM_REFUSED_DTYPE;
+#undef LAUNCH
+    return launch_status();
+}

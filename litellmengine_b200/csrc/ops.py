@@ -142,19 +142,22 @@ def _i32(t: Optional[torch.Tensor], what: str) -> None:
 # ------------------------------------------------------------------------------------------
 def embedding(ids: torch.Tensor, table: torch.Tensor, status: torch.Tensor,
               out: Optional[torch.Tensor] = None, feedback: Optional[torch.Tensor] = None,
-              scale: float = 1.0) -> torch.Tensor:
-    """float32 [T, H] = table[ids] * scale; an id -1-j takes its token from feedback[j] (int32, on the device)."""
-    _dev(ids, table, status, out, feedback)
+              scale: float = 1.0, keep: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """float32 [T, H] = table[ids] * scale; an id -1-j takes its token from feedback[j] (int32, on the device).  `keep`
+    (float32 [T, H]) receives the same rows once more."""
+    _dev(ids, table, status, out, feedback, keep)
     _i32(ids, "ids")
     if feedback is not None:
         _i32(feedback, "feedback")
     T, (V, H) = ids.numel(), table.shape
     if out is None:
         out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    if keep is not None and (keep.dtype != torch.float32 or tuple(keep.shape) != (T, H)):
+        raise KernelError("keep must be float32 [tokens, hidden]")
     f = _fn("embedding", "llm_embedding_gather",
-            [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p])
+            [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p])
     _check(f(_ptr(ids), _ptr(table), _dt(table), _ptr(out), T, H, V, _ptr(status), _ptr(feedback),
-             feedback.numel() if feedback is not None else 0, float(scale), _stream()), "embedding")
+             feedback.numel() if feedback is not None else 0, float(scale), _ptr(keep), _stream()), "embedding")
     return out
 
 
@@ -266,6 +269,40 @@ def rmsnorm_add(h: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: flo
     return copy
 
 
+def rmsnorm_sandwich(h: torch.Tensor, y, post, pre, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None,
+                     join: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The step between two sublayers that are normed on both sides, in 32-bit: v = h + rmsnorm(y) * w_post (+ join),
+    written back into the float32 stream h unless `rows` picks rows, returned as rmsnorm(v) * w_pre in `out_dtype`.
+    `post` = (w_post float32 [H], eps) or None (y joins as it is); `pre` = (w_pre float32 [H], eps).  y: None, a matrix
+    [T, H] (float32 or bfloat16), or a `PartialSum` whose k-splits are added as they are read.  `join`: float32 [T, H]."""
+    parts, part_stride = 1, 0
+    if isinstance(y, PartialSum):
+        parts, part_stride = y.parts.shape[0], y.parts.stride(0)
+        y = y.parts[0]
+    _dev(h, rows, join, pre[0], post[0] if post is not None else None)
+    _i32(rows, "rows")
+    if h.dtype != torch.float32 or h.dim() != 2:
+        raise KernelError("rmsnorm_sandwich wants a float32 stream [T, H]")
+    T, H = h.shape
+    if y is not None and (not y.is_cuda or tuple(y.shape) != (T, H) or y.stride(1) != 1):
+        raise KernelError("y must be a CUDA matrix of the stream's shape with unit stride along its rows")
+    if join is not None and (join.dtype != torch.float32 or join.shape != h.shape):
+        raise KernelError("what joins the stream must be float32 of its shape")
+    for norm in (post, pre):
+        if norm is not None and (norm[0].dtype != torch.float32 or norm[0].numel() != H):
+            raise KernelError("norm weight must be float32 of the row length")
+    n = rows.numel() if rows is not None else T
+    out = torch.empty((n, H), dtype=out_dtype, device=h.device)
+    w_post, eps_post = post if post is not None else (None, 0.0)
+    f = _fn("norm", "llm_rmsnorm_sandwich",
+            [c_void_p, c_void_p, c_int, c_longlong, c_int, c_longlong, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p,
+             c_int, c_void_p, c_int, c_int, c_void_p])
+    _check(f(_ptr(h), _ptr(y), _dt(y) if y is not None else 0, y.stride(0) if y is not None else 0, parts, part_stride,
+             _ptr(w_post), float(eps_post), _ptr(join), _ptr(pre[0]), float(pre[1]), _ptr(out), _dt(out), _ptr(rows), n, H,
+             _stream()), "rmsnorm_sandwich")
+    return out
+
+
 def tanh_norm(h: torch.Tensor, y, post, pre, out_dtype: Optional[torch.dtype] = None,
               rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """The elementwise norm n(v) = tanh(alpha v) * w + b around a residual add, in 32-bit: v = h + post(y) (written back
@@ -303,12 +340,14 @@ def tanh_norm(h: torch.Tensor, y, post, pre, out_dtype: Optional[torch.dtype] = 
     return out
 
 
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}      # the last one takes a limit
 
 
-def silu_and_mul(gate_up, out: Optional[torch.Tensor] = None, activation: str = "silu") -> torch.Tensor:
-    """[T, 2I] -> [T, I]: act(first half) * second half, act = silu or the tanh form of gelu.  A `PartialSum` is
-    added up on the way."""
+def silu_and_mul(gate_up, out: Optional[torch.Tensor] = None, activation: str = "silu",
+                 limit: float = 0.0) -> torch.Tensor:
+    """[T, 2I] -> [T, I]: act(first half) * second half, act = silu or the tanh form of gelu; 'clamped_swish':
+    g * sigmoid(1.702 g) * (u + 1) with g = min(first half, limit), u = the second half clamped to +-limit.  A
+    `PartialSum` is added up on the way."""
     act = ACTIVATIONS[activation]
     if isinstance(gate_up, PartialSum):
         parts = gate_up.parts
@@ -316,16 +355,17 @@ def silu_and_mul(gate_up, out: Optional[torch.Tensor] = None, activation: str = 
         S, T, two_i = parts.shape
         if out is None:
             out = torch.empty((T, two_i // 2), dtype=gate_up.rounds_to or torch.float32, device=parts.device)
-        f = _fn("activation", "llm_silu_and_mul_parts", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-        _check(f(_ptr(parts), S, _ptr(out), _dt(out), T, two_i // 2, act, _stream()), "silu_and_mul")
+        f = _fn("activation", "llm_silu_and_mul_parts", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                                                          c_void_p])
+        _check(f(_ptr(parts), S, _ptr(out), _dt(out), T, two_i // 2, act, float(limit), _stream()), "silu_and_mul")
         return out
     _dev(gate_up, out)
     T, two_i = gate_up.shape
     inter = two_i // 2
     if out is None:
         out = torch.empty((T, inter), dtype=gate_up.dtype, device=gate_up.device)
-    f = _fn("activation", "llm_silu_and_mul", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(f(_ptr(gate_up), _ptr(out), _dt(gate_up), T, inter, act, _stream()), "silu_and_mul")
+    f = _fn("activation", "llm_silu_and_mul", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _check(f(_ptr(gate_up), _ptr(out), _dt(gate_up), T, inter, act, float(limit), _stream()), "silu_and_mul")
     return out
 
 
@@ -1097,7 +1137,8 @@ def stream_norm(streams: torch.Tensor, y, mix: Optional[torch.Tensor], outw: Opt
 # ---- routed experts ----------------------------------------------------------------------------------------
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, groups, route_scale: float, lists: bool = False,
               score: str = "sigmoid", correction: Optional[torch.Tensor] = None, identity: int = 0,
-              bias: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None):
+              bias: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None,
+              normalize: bool = True):
     """Per token of x [T, W]: scores of `w_router` (float32 [E, W]; `score` 'sigmoid', or 'softmax' over all E), the
     `top` best among the experts of the best groups (`groups` = (count, keep) or None), weights normalised and
     scaled.  `correction` (float32 [E]) is added to the scores for the choice only.  The last `identity` router
@@ -1105,7 +1146,8 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, groups, route_s
     float32 weights [T, E - identity] (zero where not chosen) and, with `lists`, ids int32 [T, top] (-1 for an
     identity pick) and weights float32 [T, top]; with `identity`, also the float32 [T] share of a token's own input.
     `bias` (float32 [E]) joins the logits before the score.  `shared_gate` (float32 [W]): the sigmoid of its product with
-    the token comes back too, as the last member, float32 [T] (the weight of an expert that every token runs)."""
+    the token comes back too, as the last member, float32 [T] (the weight of an expert that every token runs).
+    `normalize` False: the weights are the chosen scores times `route_scale`, not divided by their sum."""
     _dev(x, w_router, correction, bias, shared_gate)
     T, W = x.shape
     E = w_router.shape[0]
@@ -1127,10 +1169,10 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, groups, route_s
     count, keep = groups if groups is not None else (0, 0)
     f = _fn("moe", "llm_moe_route",
             [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-             c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
+             c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(f(_ptr(x), _dt(x), _ptr(w_router), _ptr(dense), _ptr(ids), _ptr(wts), T, W, E, top, count, keep,
              float(route_scale), 1 if score == "softmax" else 0, _ptr(correction), identity, _ptr(idw), _ptr(bias),
-             _ptr(shared_gate), _ptr(share), _stream()), "moe_route")
+             _ptr(shared_gate), _ptr(share), 1 if normalize else 0, _stream()), "moe_route")
     out = ((dense, ids, wts) if lists else (dense,)) + ((idw,) if identity else ()) + ((share,) if share is not None else ())
     return out if len(out) > 1 else dense
 
@@ -1157,8 +1199,9 @@ def moe_finish(out: torch.Tensor, x: Optional[torch.Tensor], idw: Optional[torch
 
 
 def moe_act(gate_up, dense: Optional[torch.Tensor], E: int, ff: int, limit: float, alpha: float,
-            out_dtype: torch.dtype, shift: float = 1.0, shared=None) -> torch.Tensor:
-    """`shared` = (ff_s, limit_s, share): the rows of the product go on with a shared expert's 2 * ff_s columns, and those of
+            out_dtype: torch.dtype, shift: float = 1.0, shared=None, on_input: bool = False) -> torch.Tensor:
+    """`on_input`: a routed expert's weight multiplies its gate and up values (its input, that is) instead of its output.
+    `shared` = (ff_s, limit_s, share): the rows of the product go on with a shared expert's 2 * ff_s columns, and those of
     the result with its ff_s activations, times share[t] (float32 [T], None: one); E may then be 0.
     act [T, E*ff] = dense[t, e] * g * sigmoid(alpha g) * (u + shift), g = min(gate, limit), u = clamp(up, +-limit),
     from the float32 product [T, E*2*ff] (per expert: ff gate columns, then ff up columns; may be a `PartialSum`)."""
@@ -1176,17 +1219,17 @@ def moe_act(gate_up, dense: Optional[torch.Tensor], E: int, ff: int, limit: floa
     act = torch.empty((T, E * ff + ffs), dtype=out_dtype, device=gate_up.device)
     f = _fn("moe", "llm_moe_act",
             [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_float,
-             c_void_p, c_void_p])
+             c_void_p, c_int, c_void_p])
     _check(f(_ptr(gate_up), parts, part_stride, _ptr(dense), _ptr(act), _dt(act), T, E, ff, float(limit), float(alpha),
-             float(shift), ffs, float(limit_s), _ptr(share), _stream()), "moe_act")
+             float(shift), ffs, float(limit_s), _ptr(share), 1 if on_input else 0, _stream()), "moe_act")
     return act
 
 
 def moe_sparse(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-               ff: int, limit: float, alpha: float, shift: float = 1.0) -> torch.Tensor:
+               ff: int, limit: float, alpha: float, shift: float = 1.0, on_input: bool = False) -> torch.Tensor:
     """The routed feed-forward for steps of few tokens: only the chosen experts' matrices are read.  x [T, W] and
     the matrices in one dtype (bfloat16 or float32); `ids`, `weights` [T, top] from `moe_route`.  Returns the
-    float32 sum [T, W] of the chosen experts' weighted outputs."""
+    float32 sum [T, W] of the chosen experts' weighted outputs (`on_input`: of their outputs for the weighted input)."""
     _dev(x, w_gate_up, ids, weights)
     _i32(ids, "ids")
     T, W = x.shape
@@ -1199,9 +1242,9 @@ def moe_sparse(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, i
     out = torch.empty((T, W), dtype=torch.float32, device=x.device)
     f = _fn("moe", "llm_moe_sparse",
             [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-             c_int, c_float, c_float, c_float, c_longlong, c_void_p])
+             c_int, c_float, c_float, c_float, c_longlong, c_int, c_void_p])
     code = f(_ptr(x), _dt(x), _ptr(w_gate_up), _ptr(w_down), _dt(w_down), _ptr(ids), _ptr(weights), _ptr(act), _ptr(out),
-             T, W, ff, E, top, float(limit), float(alpha), float(shift), w_down.stride(0), _stream())
+             T, W, ff, E, top, float(limit), float(alpha), float(shift), w_down.stride(0), 1 if on_input else 0, _stream())
     _check(code, "moe_sparse")
     global launch_count
     launch_count += 1                      # two kernels in one call
@@ -1214,8 +1257,9 @@ def grouped_product_available() -> bool:
 
 
 def moe_sorted(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-               E: int, ff: int, limit: float, alpha: float, shift: float = 1.0, base: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """`base` (float32 [T, W]): the sums start from it.  The routed feed-forward for prompt portions: the (token, choice) pairs are sorted by expert (the engine's
+               E: int, ff: int, limit: float, alpha: float, shift: float = 1.0, base: Optional[torch.Tensor] = None,
+               on_input: bool = False) -> torch.Tensor:
+    """`base` (float32 [T, W]): the sums start from it.  `on_input`: the routing weight multiplies an expert's input.  The routed feed-forward for prompt portions: the (token, choice) pairs are sorted by expert (the engine's
     kernels), each expert's rows go through ITS matrices in the library's grouped matrix product (bfloat16 in,
     bfloat16 out, 32-bit accumulation; the row offsets stay on the device), the activation takes each row's
     routing weight, and a token's rows are added in 32-bit.  Returns float32 [T, W]."""
@@ -1232,16 +1276,16 @@ def moe_sorted(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, i
     _check(_fn("moe", "llm_moe_sort", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])(
         _ptr(ids), pairs, E, _ptr(offs), _ptr(pos), _ptr(row_pair), _stream()), "moe_sort")
     rows_fn = _fn("moe", "llm_moe_rows",
-                  [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p])
+                  [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p])
     xs = torch.empty((pairs, W), dtype=x.dtype, device=dev)
-    _check(rows_fn(0, _ptr(x), _dt(x), _ptr(row_pair), None, _ptr(xs), pairs, W, top, 0.0, 0.0, 0.0, _stream()), "moe_gather")
+    _check(rows_fn(0, _ptr(x), _dt(x), _ptr(row_pair), None, _ptr(xs), pairs, W, top, 0.0, 0.0, 0.0, 0, _stream()), "moe_gather")
     gu = torch._grouped_mm(xs, w_gate_up.view(E, 2 * ff, W).transpose(1, 2), offs=offs)
     act = torch.empty((pairs, ff), dtype=x.dtype, device=dev)
     _check(rows_fn(1, _ptr(gu), _dt(gu), _ptr(row_pair), _ptr(weights), _ptr(act), pairs, ff, top, float(limit), float(alpha),
-                   float(shift), _stream()), "moe_act_pairs")
+                   float(shift), 1 if on_input else 0, _stream()), "moe_act_pairs")
     y = torch._grouped_mm(act, w_down.as_strided((E, ff, W), (ff, 1, w_down.stride(0)), w_down.storage_offset()), offs=offs)
     out = torch.empty((T, W), dtype=torch.float32, device=dev)
-    _check(rows_fn(2, _ptr(y), _dt(y), _ptr(pos), _ptr(base), _ptr(out), T, W, top, 0.0, 0.0, 0.0, _stream()), "moe_combine")
+    _check(rows_fn(2, _ptr(y), _dt(y), _ptr(pos), _ptr(base), _ptr(out), T, W, top, 0.0, 0.0, 0.0, 0, _stream()), "moe_combine")
     return out
 
 
@@ -1666,8 +1710,8 @@ def linear_pair(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype,
 
 
 def linear_pair_silu_mul(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None,
-                         activation: str = "silu") -> torch.Tensor:
-    """act(x @ gate^T) * (x @ up^T), act = silu or the tanh form of gelu, for w_gate_up = [gate; up] of 2 I rows, as bfloat16 [T, I]: the
+                         activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
+    """act(x @ gate^T) * (x @ up^T), act as in `silu_and_mul`, for w_gate_up = [gate; up] of 2 I rows, as bfloat16 [T, I]: the
     paired tcgen05 product with the activation in its epilogue (gate and up are rounded to bfloat16
     before the activation, as the separate kernel would read them)."""
     _dev(x, w_gate_up, out)
@@ -1679,9 +1723,9 @@ def linear_pair_silu_mul(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional
     inter = w_gate_up.shape[0] // 2
     if out is None:
         out = torch.empty((T, inter), dtype=torch.bfloat16, device=x.device)
-    f = _fn("gemm_pair_tcgen05", "llm_linear_pair_silu_mul", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+    f = _fn("gemm_pair_tcgen05", "llm_linear_pair_silu_mul", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p,
                                                               c_void_p])
-    _check(f(_ptr(x), _ptr(w_gate_up), _ptr(out), T, inter, K, ACTIVATIONS[activation], _ptr(stream_status(x.device)), _stream()),
+    _check(f(_ptr(x), _ptr(w_gate_up), _ptr(out), T, inter, K, ACTIVATIONS[activation], float(limit), _ptr(stream_status(x.device)), _stream()),
            "linear_pair_silu_mul")
     return out
 
@@ -1722,12 +1766,13 @@ def linear_into(x: torch.Tensor, weight: torch.Tensor, residual: torch.Tensor) -
     return True
 
 
-def linear_silu_mul(x: torch.Tensor, w_gate_up: torch.Tensor, out_dtype: torch.dtype, activation: str = "silu"):
+def linear_silu_mul(x: torch.Tensor, w_gate_up: torch.Tensor, out_dtype: torch.dtype, activation: str = "silu",
+                    limit: float = 0.0):
     """act(x @ gate^T) * (x @ up^T) for w_gate_up = [gate; up]: one kernel where the paired product
     takes it, else the product (which may stay a sum of k-splits) followed by the activation kernel."""
     if out_dtype == torch.bfloat16 and _pair_takes(x, w_gate_up, w_gate_up.shape[0] // 2, "silu"):
-        return linear_pair_silu_mul(x, w_gate_up, activation=activation)
-    return silu_and_mul(linear(x, w_gate_up, out_dtype=out_dtype, partials_ok=True), activation=activation)
+        return linear_pair_silu_mul(x, w_gate_up, activation=activation, limit=limit)
+    return silu_and_mul(linear(x, w_gate_up, out_dtype=out_dtype, partials_ok=True), activation=activation, limit=limit)
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,

@@ -86,8 +86,7 @@ class AttentionMixer:
             raise ValueError("attention heads must be a positive multiple of kv heads")
         if spec.head_dim <= 0 or spec.head_dim % 16 or spec.head_dim > 256:
             raise ValueError(f"head_dim {spec.head_dim}: the attention kernels take multiples of 16 up to 256")
-        if spec.window is not None and spec.window <= 0:
-            raise ValueError("an attention window must be positive")
+        self.span = key_span(spec)
         self.spec = spec
         self.hidden = hidden_size
         self.nq, self.nkv, self.d = spec.num_heads, spec.num_kv_heads, spec.head_dim
@@ -134,14 +133,14 @@ class AttentionMixer:
     def cache_need(self):
         if not self.spec.has_kv:
             return None
-        return PagedNeed(self.nkv, self.d, self.spec.window)
+        return PagedNeed(self.nkv, self.d, self.spec.window, chunk=self.spec.chunk)
 
     def step_prelude(self):
         return AttentionWork()
 
     @property
     def graph_variant_group(self):
-        return ("attention", self.nkv)
+        return ("attention", self.nkv, self.span)
 
     def graph_variant(self, batch, padded: bool) -> int:
         """The decode kernel's key splits: the one launch choice here that depends on lengths."""
@@ -149,7 +148,7 @@ class AttentionMixer:
         if work is None:
             return 0
         n_dec = work.padded_rows.shape[0] if padded else work.num_decode
-        return decode_key_splits(self.device, n_dec, self.nkv, batch.max_kv_len) if n_dec else 0
+        return decode_key_splits(self.device, n_dec, self.nkv, decode_reach(batch, self.span)) if n_dec else 0
 
     def forward(self, x: torch.Tensor, ctx: StageContext) -> torch.Tensor:
         b = ctx.batch
@@ -179,7 +178,7 @@ class AttentionMixer:
                              k32.reshape(T, self.nkv * self.d).contiguous() if k32 is not None else None, qkv, cache,
                              b.positions, b.token_entry, b.entry_slot, table, self.nq, self.nkv, self.d,
                              ctx.page_size, has_kv, ctx.status, self.dtype)
-        a = attention_over_pages(q, ctx, self.nq, self.nkv, self.d, self.spec.window, self.scale)
+        a = attention_over_pages(q, ctx, self.nq, self.nkv, self.d, self.span, self.scale)
         # joins the float32 residual; may stay a sum of k-splits if the layer's norm adds them itself
         residual = getattr(ctx, "residual", None)
         if residual is not None and ops.linear_into(a, self.w_o, residual):
@@ -221,7 +220,7 @@ class GatedAttentionMixer(BranchMixer):
     values of their own width, biased q/k/v projections, a q/k norm per head or over the token's whole
     projection, a query temperature q *= 1 + coef * ln(floor((p + 1) / every) + 1), and an output gate
     sigmoid(W_g x) on the concatenated heads before the output projection.  Rotations of either pair layout; a
-    window that keeps the sequence's first keys; a softmax sink, one constant or a learned score per head.  One product yields [q | k | v | g] per token in
+    window that keeps the sequence's first keys, or chunks; a softmax sink, one constant or a learned score per head.  One product yields [q | k | v | g] per token in
     float32; one kernel adds the biases, normalises, applies the temperature and writes keys and values
     to their pages; the attention kernel applies the gate as it stores.  The gate may be one value per head
     (`output_gate_scope` 'head').  `distance_bias` = (rows, far) adds a learned bias table[bucket(i - j), head]
@@ -254,8 +253,7 @@ class GatedAttentionMixer(BranchMixer):
             raise ValueError("the gated attention mixer keeps its own keys and values")
         if spec.output_gate_scope not in ("channel", "head"):
             raise ValueError(f"output_gate_scope {spec.output_gate_scope!r}: 'channel' or 'head'")
-        if spec.window is not None and spec.window <= 0:
-            raise ValueError("an attention window must be positive")
+        self.span = key_span(spec)
         self.spec, self.hidden, self.dtype, self.device = spec, hidden_size, compute_dtype, torch.device(device)
         self.nq, self.nkv, self.d = spec.num_heads, spec.num_kv_heads, spec.head_dim
         self.scale = spec.scale if spec.scale is not None else 1.0 / math.sqrt(float(self.d))
@@ -361,8 +359,8 @@ class GatedAttentionMixer(BranchMixer):
                 raise ValueError("distance_bias: the farthest distance must exceed half the number of rows")
             # from distance ceil(far) on the row no longer changes; a window never asks beyond its size
             count = int(math.ceil(far)) + 1
-            if s.window is not None:
-                count = min(count, s.window)
+            if self.span is not None:
+                count = min(count, abs(self.span))
             index = torch.tensor([distance_bucket(d, rows, far) for d in range(count)], dtype=torch.long, device=rel.device)
             self.dist_table = rel[index].contiguous()
             # for the tensor-core kernel: a row per head, in the exp2 domain
@@ -371,18 +369,15 @@ class GatedAttentionMixer(BranchMixer):
         ops.prepare_streaming(self.w_o)
 
     def cache_need(self):
-        return PagedNeed(self.nkv, self.d, self.spec.window, None if self.dv == self.d else self.dv, self.keep_first)
+        return PagedNeed(self.nkv, self.d, self.spec.window, None if self.dv == self.d else self.dv, self.keep_first,
+                         self.spec.chunk)
 
     def step_prelude(self):
         return AttentionWork() if self._tuned or self._tuned_prompt else None
 
     @property
     def graph_variant_group(self):
-        return ("attention", self.nkv) if self._tuned else ("gated_attention", self.nkv, self.spec.window)
-
-    def _decode_reach(self, batch) -> int:
-        """The most keys a single token of this step walks: the longest cached length, or the window."""
-        return min(batch.max_kv_len, self.spec.window) if self.spec.window else batch.max_kv_len
+        return ("attention" if self._tuned else "gated_attention", self.nkv, self.span)
 
     def graph_variant(self, batch, padded: bool) -> int:
         if self._tuned:
@@ -392,7 +387,7 @@ class GatedAttentionMixer(BranchMixer):
         work = batch.preludes.get(AttentionWork.name)       # the decode kernel's key splits, as the step will choose them
         n_dec = 0 if work is None else (work.padded_rows.shape[0] if padded else work.num_decode)
         n_tiles = 0 if work is None else (work.padded_tiles.shape[0] if padded else work.num_prefill_tiles)
-        return decode_key_splits(self.device, n_dec, self.nkv, self._decode_reach(batch)) if n_dec and not n_tiles else 0
+        return decode_key_splits(self.device, n_dec, self.nkv, decode_reach(batch, self.span)) if n_dec and not n_tiles else 0
 
     def mix(self, proj, col0, ctx, out, out_col0, out_scale):
         b, s = ctx.batch, self.spec
@@ -405,8 +400,12 @@ class GatedAttentionMixer(BranchMixer):
             ctx.block_table, self.nq, self.nkv, self.d, self.dv, ctx.page_size, ctx.status, self.dtype,
             rotation=self.rotation)
         if self._tuned and ctx.cache is not None and b.preludes.get(AttentionWork.name) is not None:
-            a = attention_over_pages(q, ctx, self.nq, self.nkv, self.d, s.window, self.scale)
-            ops.gate_mul(a, proj, col0 + self.g_off, out, out_col0, s.output_gate, out_scale)
+            # without a gate, a scale or a column offset the kernels write where the output product reads
+            direct = (not s.output_gate and out_col0 == 0 and out_scale == 1.0 and out.is_contiguous()
+                      and tuple(out.shape) == tuple(q.shape))
+            a = attention_over_pages(q, ctx, self.nq, self.nkv, self.d, self.span, self.scale, out=out if direct else None)
+            if not direct:
+                ops.gate_mul(a, proj, col0 + self.g_off, out, out_col0, s.output_gate, out_scale)
             return
         work = b.preludes.get(AttentionWork.name) if self._tuned_prompt and ctx.cache is not None else None
         padded = getattr(b, "any_division", False)
@@ -424,12 +423,12 @@ class GatedAttentionMixer(BranchMixer):
                 ops.paged_attention_prefill_tcgen05_biased(
                     q, out, ctx.cache, work.padded_tiles if padded else work.prefill_tiles, n_tiles, b.entry_slot,
                     b.entry_q_start, b.entry_q_len, b.entry_kv_len, ctx.block_table, self.nq, self.nkv, self.d,
-                    ctx.page_size, s.window, self.scale, ctx.status, self.dist_table_t)
+                    ctx.page_size, self.span, self.scale, ctx.status, self.dist_table_t)
             elif n_tiles:
                 ops.paged_attention_prefill_biased(
                     q, out, out_col0, ctx.cache, work.padded_tiles if padded else work.prefill_tiles, n_tiles, b.entry_slot,
                     b.entry_q_start, b.entry_q_len, b.entry_kv_len, ctx.block_table, self.nq, self.nkv, self.d, ctx.page_size,
-                    s.window, self.scale, ctx.status, dist_bias_t=self.dist_table_t, head_gate=gate,
+                    self.span, self.scale, ctx.status, dist_bias_t=self.dist_table_t, head_gate=gate,
                     gate_off=col0 + self.g_off, out_scale=out_scale, analytic_bias=self.analytic,
                     keep_first=self.keep_first, sink=self.sink)
             if not n_dec:
@@ -440,9 +439,9 @@ class GatedAttentionMixer(BranchMixer):
                 direct = (gate is None and out_col0 == 0 and out_scale == 1.0 and out.is_contiguous()
                           and tuple(out.shape) == tuple(q.shape))
                 a = out if direct else torch.empty_like(q)
-                splits = decode_key_splits(q.device, n_dec, self.nkv, self._decode_reach(b))
+                splits = decode_key_splits(q.device, n_dec, self.nkv, decode_reach(b, self.span))
                 ops.paged_attention_decode(q, a, ctx.cache, rows, n_dec, b.positions, b.token_entry, b.entry_slot,
-                                           ctx.block_table, self.nq, self.nkv, self.d, ctx.page_size, s.window, self.scale, splits,
+                                           ctx.block_table, self.nq, self.nkv, self.d, ctx.page_size, self.span, self.scale, splits,
                                            ctx.status, dist_bias_t=self.dist_table_t, analytic_bias=self.analytic,
                                            keep_first=self.keep_first, sink=self.sink)
                 if not direct:
@@ -453,7 +452,7 @@ class GatedAttentionMixer(BranchMixer):
             rows = None
         ops.paged_attention_generic_kv(
             q, ctx.cache_keys, ctx.cache_values, b.positions, b.token_entry, b.entry_slot, ctx.block_table, self.nq,
-            self.nkv, self.d, self.dv, ctx.page_size, s.window, self.scale, ctx.status, out, out_col0,
+            self.nkv, self.d, self.dv, ctx.page_size, self.span, self.scale, ctx.status, out, out_col0,
             gate=proj if s.output_gate else None, gate_off=col0 + self.g_off, out_scale=out_scale,
             dist_bias=self.dist_table, gate_per_head=self.gate_per_head, rows=rows, head_scale=self.head_temp,
             log_bias=(self.log_r1, self.log_r2) if self.log_r1 is not None else None, keep_first=self.keep_first,
@@ -467,6 +466,21 @@ def distance_bucket(n: int, rows: int, far: float) -> int:
     if n < half:
         return n
     return min(rows - 1, half + int(math.floor(math.log(n / half) / math.log(far / half) * (rows - half))))
+
+
+def key_span(spec: MixerSpec) -> Optional[int]:
+    """Which keys a query sees, as the kernels take it (their `window`): w > 0, the last w; -c, those of its own chunk of c
+    positions; None, all."""
+    if spec.window is not None and spec.window <= 0:
+        raise ValueError("an attention window must be positive")
+    if spec.chunk is not None and (spec.chunk <= 0 or spec.window is not None):
+        raise ValueError("an attention chunk must be positive and excludes a window")
+    return -spec.chunk if spec.chunk is not None else spec.window
+
+
+def decode_reach(batch, span: Optional[int]) -> int:
+    """The most keys a single token of this step walks: the longest cached length, at most the window or the chunk."""
+    return min(batch.max_kv_len, abs(span)) if span else batch.max_kv_len
 
 
 _slots = {}
@@ -510,35 +524,36 @@ _split_choice: Dict[tuple, int] = {}
 
 
 def attention_over_pages(q: torch.Tensor, ctx: StageContext, nq: int, nkv: int, d: int,
-                         window: Optional[int], scale: float) -> torch.Tensor:
+                         span: Optional[int], scale: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Pick the attention kernels for this batch.  Every choice reads the same pages and gives
     the same result up to rounding.  bfloat16 with a head size and group the tuned kernels
     take: single tokens go to the split-key decode kernel, longer portions to the tensor-core
     prefill kernel (a mixed batch launches both, each over its own rows).  Everything else,
-    float32 included, goes through the generic kernel."""
+    float32 included, goes through the generic kernel.  `span`: see `key_span`.  `out`: where the result goes, if the
+    tuned kernels take the step (bfloat16 [T, heads * head_dim], contiguous)."""
     b = ctx.batch
     cache = ctx.cache
     work = b.preludes.get(AttentionWork.name)
     if (work is not None and q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16
             and ops.fast_attention_supported(d, nq // nkv)):
-        out = torch.empty_like(q)
+        out = torch.empty_like(q) if out is None else out
         # A step that is being captured as a graph of "any step of this many tokens" launches both
         # kernels over the padded lists; otherwise over what this step has.
         padded = getattr(b, "any_division", False)
         n_dec = work.padded_rows.shape[0] if padded else work.num_decode
         n_tiles = work.padded_tiles.shape[0] if padded else work.num_prefill_tiles
         if n_dec:
-            splits = decode_key_splits(q.device, n_dec, nkv, b.max_kv_len)
+            splits = decode_key_splits(q.device, n_dec, nkv, decode_reach(b, span))
             rows = work.padded_rows if padded else (None if n_dec == b.num_tokens else work.decode_rows)
             ops.paged_attention_decode(q, out, cache, rows, n_dec, b.positions, b.token_entry, b.entry_slot,
-                                       ctx.block_table, nq, nkv, d, ctx.page_size, window, scale, splits, ctx.status)
+                                       ctx.block_table, nq, nkv, d, ctx.page_size, span, scale, splits, ctx.status)
         if n_tiles:
             kernel = (ops.paged_attention_prefill_tcgen05
                       if ops.prefill_tcgen05_supported(d, ctx.page_size)
                       else ops.paged_attention_prefill)       # tcgen05/TMEM/TMA where it applies, mma.sync otherwise
             kernel(q, out, cache, work.padded_tiles if padded else work.prefill_tiles, n_tiles, b.entry_slot,
-                   b.entry_q_start, b.entry_q_len, b.entry_kv_len, ctx.block_table, nq, nkv, d, ctx.page_size, window,
+                   b.entry_q_start, b.entry_q_len, b.entry_kv_len, ctx.block_table, nq, nkv, d, ctx.page_size, span,
                    scale, ctx.status)
         return out
     return ops.paged_attention_generic(q, cache, b.positions, b.token_entry, b.entry_slot,
-                                       ctx.block_table, nq, nkv, d, ctx.page_size, window, scale, ctx.status)
+                                       ctx.block_table, nq, nkv, d, ctx.page_size, span, scale, ctx.status)

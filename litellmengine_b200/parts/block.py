@@ -80,6 +80,20 @@ class InputConvolution:
         return ops.short_conv(x, self.weight, kept, batch, out_dtype)
 
 
+class LayerScale:
+    """A learned factor per channel on a sublayer's normed output (tensor [hidden])."""
+
+    def __init__(self, size: int):
+        self.size = size
+        self.weight: Optional[torch.Tensor] = None
+
+    def parameters(self) -> Dict[str, ParamSpec]:
+        return {"": ParamSpec((self.size,), role="scale", init=("one_plus_normal", 0.1))}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = tensors[""].contiguous()
+
+
 class Block:
     """Holds one layer's mixer, feed-forward and norms, each chosen by the layer's spec."""
 
@@ -106,6 +120,15 @@ class Block:
             self.mixer_post_norm = lookup("norm", spec.mixer_post_norm.kind)(spec.mixer_post_norm, hidden_size)
         if getattr(spec, "feed_forward_post_norm", None) is not None and spec.feed_forward is not None:
             self.feed_forward_post_norm = lookup("norm", spec.feed_forward_post_norm.kind)(spec.feed_forward_post_norm, hidden_size)
+        # what multiplies a sublayer's normed output: it joins the weight of the norm on that output
+        self.branch_scale = float(getattr(spec, "branch_scale", 1.0))
+        self.layer_scales = None
+        if getattr(spec, "layer_scale_names", None) is not None:
+            self.layer_scales = (LayerScale(hidden_size), LayerScale(hidden_size) if self.feed_forward is not None else None)
+        if self.layer_scales is not None or self.branch_scale != 1.0:
+            for norm in self._output_norms():
+                if not hasattr(norm, "scale_output"):
+                    raise ValueError("a factor on the sublayers' outputs needs norms there that take it")
         self.arrangement = lookup("arrangement", spec.arrangement)
         # a model with several residual streams: one connection per sublayer
         self.connections = None
@@ -120,6 +143,9 @@ class Block:
                                 InputConvolution(hidden_size, taps) if self.feed_forward is not None else None)
         self.residual_scale = float(getattr(spec, "residual_scale", 1.0))
         self.hidden = hidden_size
+
+    def _output_norms(self):
+        return [self.mixer_post_norm] + ([self.feed_forward_post_norm] if self.feed_forward is not None else [])
 
     def state_need(self):
         """What the layer keeps per request beside its mixer's cache: the last taps - 1 rows of the stream in front of
@@ -144,6 +170,8 @@ class Block:
             out.append((s.feed_forward_post_norm_name, self.feed_forward_post_norm))
         if self.connections is not None:
             out += [(name, c) for name, c in zip(s.connections[1:], self.connections) if c is not None]
+        if self.layer_scales is not None:
+            out += [(name, c) for name, c in zip(s.layer_scale_names, self.layer_scales) if c is not None]
         if self.input_convs is not None:
             out += [(name, c) for name, c in zip(s.input_conv_names, self.input_convs) if c is not None]
         return out
@@ -165,6 +193,9 @@ class Block:
             if prefix in tensors and "" in part.parameters():
                 mine[""] = tensors[prefix]
             part.load({n: t for n, t in mine.items() if n in part.parameters()})
+        if self.layer_scales is not None or self.branch_scale != 1.0:
+            for norm, ls in zip(self._output_norms(), self.layer_scales or (None, None)):
+                norm.scale_output(self.branch_scale if ls is None else ls.weight * self.branch_scale)
 
     def forward(self, h: torch.Tensor, delta: Optional[torch.Tensor], ctx: StageContext
                 ) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
@@ -270,7 +301,8 @@ def sandwich_norm(block: Block, h: torch.Tensor, delta, ctx: StageContext):
     """h += norm1b(mixer(norm1(h))); h += norm2b(ffn(norm2(h))): a norm in front of every sublayer and one on its
     output.  `h` is the float32 residual stream; a sublayer's output does not join it when the sublayer returns: it
     travels on (across layers too) as a `PendingNormed` with the norm of its way, and the kernel that makes the next
-    sublayer's normed input adds it as it reads.  The norms must take a `PendingNormed` as their `delta`."""
+    sublayer's normed input adds it as it reads.  The norms must take a `PendingNormed` as their `delta`.  Factors on the
+    sublayers' outputs (`layer_scale_names`, `branch_scale`) are in the output norms' weights since the layer was loaded."""
     from .norms import PendingNormed
     x = block.mixer_norm.forward(h, block.dtype, delta=delta, write_sum=delta is not None)
     ctx.partials_ok = True                                      # the norm kernel adds a product's k-splits as it reads

@@ -14,8 +14,9 @@ from .registry import register_feed_forward
 @register_feed_forward("swiglu")
 class SwiGLU:
     """down(act(gate(x)) * up(x)), no biases, act = silu (src/model/qwen3.cpp:143-152,
-    src/ops/silu_and_mul.cu:44-46) or what the spec's `params` name as `activation` ('gelu_tanh').  Gate and up are
-    one fused product [g | u]."""
+    src/ops/silu_and_mul.cu:44-46) or what the spec's `params` name as `activation` ('gelu_tanh'; 'clamped_swish':
+    down(g * sigmoid(1.702 g) * (u + 1)) with g = min(gate x, limit), u = clamp(up x, -limit, limit), `params` limit).
+    Gate and up are one fused product [g | u]."""
 
     graph_safe = True          # forward only launches kernels on the current stream
     any_division_safe = True   # and nothing in it is shaped by the number of entries of the step
@@ -30,6 +31,11 @@ class SwiGLU:
         self.activation = dict(getattr(spec, "params", ())).get("activation", "silu")
         if self.activation not in ops.ACTIVATIONS:
             raise ValueError(f"activation {self.activation!r}: one of {sorted(ops.ACTIVATIONS)}")
+        self.limit = 0.0
+        if self.activation == "clamped_swish":
+            self.limit = float(dict(spec.params)["limit"])
+            if not self.limit > 0:
+                raise ValueError("a clamped feed-forward needs a positive limit")
         self.w_gate_up: Optional[torch.Tensor] = None
         self.w_down: Optional[torch.Tensor] = None
 
@@ -50,7 +56,7 @@ class SwiGLU:
     supports_residual = True   # forward(x, residual=h) may add its result to h itself and return None
 
     def forward(self, x: torch.Tensor, partials_ok: bool = False, residual: Optional[torch.Tensor] = None):
-        act = ops.linear_silu_mul(x, self.w_gate_up, self.dtype, self.activation)
+        act = ops.linear_silu_mul(x, self.w_gate_up, self.dtype, self.activation, self.limit)
         if residual is not None and ops.linear_into(act, self.w_down, residual):
             return None                                                               # joined the residual in the product
         return ops.linear(act, self.w_down, out_dtype=torch.float32, partials_ok=partials_ok)
@@ -84,7 +90,9 @@ class RoutedExperts:
     expert of the clamped form with a limit of its own (`shared_limit`), and with `shared_gate` its output is multiplied by
     sigmoid(W_sg x), one number per token (tensor 'shared.sg' [1, hidden], applied by the router's kernel).  Such a shared
     expert's matrices lie behind the routed experts' in the same two matrices, so that the one-product form runs it as one
-    more expert."""
+    more expert.  `normalize` False: the chosen experts' weights are their scores (times route_scale) as they are, not
+    divided by their sum; `weight_on_input`: a routed expert runs on weight * x instead of having its output multiplied
+    (the gate and up products are linear in x, so the weight joins between them and the activation)."""
 
     graph_safe = True
     any_division_safe = True
@@ -108,6 +116,8 @@ class RoutedExperts:
             raise ValueError(f"activation {self.activation!r}: 'clamped_swish' or 'silu'")
         self.score = p.get("score", "sigmoid")
         self.identity = int(p.get("identity", 0) or 0)
+        self.normalize = bool(p.get("normalize", True))
+        self.on_input = bool(p.get("weight_on_input", False))
         self.has_correction = bool(p.get("correction", False))
         self.correction = None
         self.shared = None
@@ -135,6 +145,8 @@ class RoutedExperts:
             raise ValueError("routed experts need a positive size, experts and 0 < top <= the router's outputs")
         if self.score not in ("sigmoid", "softmax"):
             raise ValueError(f"score {self.score!r}: 'sigmoid' or 'softmax'")
+        if self.on_input and self.identity:
+            raise ValueError("router outputs without an expert return the input times their weight: no weight on the input beside them")
         if self.groups is not None and self.identity:
             raise ValueError("expert groups and router outputs without an expert exclude one another")
         if self.groups is not None:
@@ -190,7 +202,8 @@ class RoutedExperts:
     def _route(self, x: torch.Tensor, lists: bool):
         """(dense weights, ids, weights, the tokens' share of their own input or None, the shared expert's weights or None)."""
         got = ops.moe_route(x, self.w_router, self.top, self.groups, self.route_scale, lists=lists, score=self.score,
-                            correction=self.correction, identity=self.identity, bias=self.bias, shared_gate=self.w_sg)
+                            correction=self.correction, identity=self.identity, bias=self.bias, shared_gate=self.w_sg,
+                            normalize=self.normalize)
         got = list(got) if isinstance(got, tuple) else [got]
         share = got.pop() if self.w_sg is not None else None
         own = got.pop() if self.identity else None
@@ -212,7 +225,7 @@ class RoutedExperts:
                 and self.top * self.ff <= 12288):
             _, ids, weights, own, share = self._route(x, True)
             out = ops.moe_sparse(x, self.w_gate_up[:routed_rows], self.w_down[:, :routed_cols], ids, weights, self.ff, *act,
-                                 shift=self.act_shift)
+                                 shift=self.act_shift, on_input=self.on_input)
             if self.joined is not None:
                 joined = self._shared_alone(x, share, True)
         elif (T > self.SORTED_FROM and x.dtype == torch.bfloat16 and self.w_gate_up.dtype == self.w_down.dtype == torch.bfloat16
@@ -221,12 +234,12 @@ class RoutedExperts:
             _, ids, weights, own, share = self._route(x, True)
             base = self._shared_alone(x, share, False) if self.joined is not None else None
             out = ops.moe_sorted(x, self.w_gate_up[:routed_rows], self.w_down[:, :routed_cols], ids, weights, self.E, self.ff, *act,
-                                 shift=self.act_shift, base=base)
+                                 shift=self.act_shift, base=base, on_input=self.on_input)
         else:
             dense, _, _, own, share = self._route(x, False)
             gate_up = ops.linear(x, self.w_gate_up, out_dtype=torch.float32, partials_ok=True)
             a = ops.moe_act(gate_up, dense, self.E, self.ff, *act, self.dtype, shift=self.act_shift,
-                            shared=self.joined + (share,) if self.joined is not None else None)
+                            shared=self.joined + (share,) if self.joined is not None else None, on_input=self.on_input)
             out = ops.linear(a, self.w_down, out_dtype=torch.float32, partials_ok=partials_ok and plain)
         if plain and joined is None:
             return out

@@ -12,7 +12,7 @@ from .block import Block, streams_norm
 from .context import StageContext
 from .norms import PendingSum
 from .registry import lookup
-from .rejoin import EmbeddingRejoin
+from .rejoin import REJOINS, AddedEmbedding
 
 
 def _compute_dtype(name) -> torch.dtype:
@@ -48,7 +48,7 @@ class Model:
         self.embedding_norm = None
         if plan.embedding_norm is not None:
             self.embedding_norm = lookup("norm", plan.embedding_norm.kind)(plan.embedding_norm, plan.hidden_size)
-        self.rejoin = EmbeddingRejoin(plan.rejoin, plan.hidden_size, self.dtype) if plan.rejoin is not None else None
+        self.rejoin = REJOINS[plan.rejoin.kind](plan.rejoin, plan.hidden_size, self.dtype) if plan.rejoin is not None else None
         self.embedding: Optional[torch.Tensor] = None
         self.output: Optional[torch.Tensor] = None
 
@@ -155,8 +155,8 @@ class Model:
                     if isinstance(v, torch.Tensor) and v.dim() in (2, 3):
                         add(v)
         if self.rejoin is not None:
-            add(self.rejoin.w_x)
-            add(self.rejoin.w_e)
+            for w in self.rejoin.matrices():
+                add(w)
         add(self.output)
         return total
 
@@ -165,9 +165,10 @@ class Model:
         """batch: StepBatch already on the device; cache: CacheManager.  Returns float32
         [batch.num_want, vocab] (an empty tensor when nothing is wanted)."""
         with ops.bound_stream():                       # one stream for the whole pass, looked up once
-            copy = base = None
+            copy = base = x0 = None
+            adds = isinstance(self.rejoin, AddedEmbedding)
             if self.embedding_norm is not None:
-                norm, narrow = self.embedding_norm, self.rejoin is not None and self.dtype != torch.float32
+                norm, narrow = self.embedding_norm, self.rejoin is not None and not adds and self.dtype != torch.float32
                 h, copy = ops.embedding_norm(batch.token_ids, self.embedding, norm.weight, getattr(norm, "bias", None), norm.eps,
                                              norm.center, batch.status, feedback=getattr(batch, "feedback", None),
                                              copy_dtype=self.dtype if narrow else None)
@@ -180,16 +181,22 @@ class Model:
                 ops.embedding(batch.token_ids, self.embedding, batch.status, out=h[0],
                               feedback=getattr(batch, "feedback", None), scale=self.plan.embedding_scale)
             else:
+                if adds:
+                    x0 = torch.empty((batch.num_tokens, self.plan.hidden_size), dtype=torch.float32, device=self.device)
                 h = ops.embedding(batch.token_ids, self.embedding, batch.status, feedback=getattr(batch, "feedback", None),
-                                  scale=self.plan.embedding_scale)
-            if self.rejoin is not None:                # what every pass of the looped span starts from
+                                  scale=self.plan.embedding_scale, keep=x0)
+            if adds:
+                x0 = h.clone() if x0 is None else x0   # the stream is written in place
+            elif self.rejoin is not None:              # what every pass of the looped span starts from
                 if copy is None:
                     copy = h if self.dtype == torch.float32 else h.to(self.dtype)
                 base = self.rejoin.begin(copy)
             delta = None
             for s, st in enumerate(self.plan.order):
                 block = self.blocks[st.block]
-                if st.starts_pass is not None:
+                if st.starts_pass is not None and adds:
+                    delta = self.rejoin.start(h, delta, x0, st.starts_pass, block.mixer_norm)
+                elif st.starts_pass is not None:
                     delta = self.rejoin.start(h, copy if s == 0 else None, delta, base, st.starts_pass)
                     if not getattr(block.mixer_norm, "accepts_pending", False):
                         delta.settle_into(h)

@@ -14,9 +14,12 @@ from .registry import register_norm
 @register_norm("rmsnorm")
 class RMSNorm:
     """out = v * rsqrt(mean(v^2) + eps) * weight with v = x (+ delta), everything in 32-bit
-    (src/layers/rms_norm.cu:77-93).  The weight multiplies directly (no 1 + w)."""
+    (src/layers/rms_norm.cu:77-93).  The weight multiplies directly (no 1 + w).  `delta` may be a `PendingNormed`: a
+    sublayer's output and the norm of this kind that it passes before it joins the stream, which the same kernel
+    applies, with whatever else joins there; the sum is then written back into x unless `rows` picks rows."""
 
     accepts_partials = True    # `delta` may be an ops.PartialSum: the kernel adds the k-splits as it reads
+    accepts_join = True        # and a PendingNormed with a `join`
     center = False             # what a kernel that applies this norm itself needs to know beside weight and eps
 
     def __init__(self, spec: NormSpec, size: int):
@@ -31,6 +34,10 @@ class RMSNorm:
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.weight = tensors[self.name].contiguous()
 
+    def scale_output(self, factor) -> None:
+        """From now on the norm's output is multiplied by `factor` (a number, or float32 [size]): it joins the weight."""
+        self.weight = (self.weight * factor).contiguous()
+
     def add_normed(self, h: torch.Tensor, y, copy_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
         """h += norm(y) * weight in place (the norm of a sublayer's OUTPUT joined with the residual add);
         returns the new h in `copy_dtype` if one is asked for."""
@@ -38,6 +45,12 @@ class RMSNorm:
 
     def forward(self, x: torch.Tensor, out_dtype: torch.dtype, delta: Optional[torch.Tensor] = None,
                 rows: Optional[torch.Tensor] = None, write_sum: bool = False) -> torch.Tensor:
+        if isinstance(delta, PendingNormed):
+            y = delta.y
+            if isinstance(y, ops.PartialSum) and y.rounds_to is not None:
+                y = ops.as_tensor(y)                 # k-splits of a product that is not 32-bit: their sum is rounded first
+            post = (delta.norm.weight, delta.norm.eps) if delta.norm is not None else None
+            return ops.rmsnorm_sandwich(x, y, post, (self.weight, self.eps), out_dtype, rows=rows, join=delta.join)
         return ops.rmsnorm(x, self.weight, self.eps, out_dtype, delta=delta, rows=rows, write_sum=write_sum)
 
 
@@ -117,10 +130,11 @@ class PendingStart:
 
 class PendingNormed:
     """A sublayer's output that has not joined the residual stream yet, with the norm it passes on its way there
-    (None: it joins as it is).  The kernel that norms the next sublayer's input applies both on the way."""
+    (None: it joins as it is).  The kernel that norms the next sublayer's input applies both on the way.  `join`
+    (float32, the stream's shape): one more summand that joins there, for norms with `accepts_join`."""
 
-    def __init__(self, y, norm=None):
-        self.y, self.norm = y, norm
+    def __init__(self, y, norm=None, join: Optional[torch.Tensor] = None):
+        self.y, self.norm, self.join = y, norm, join
 
 
 @register_norm("tanh")

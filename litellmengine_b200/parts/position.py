@@ -112,7 +112,8 @@ class PairRotation:
     angle float(position) * freq[i]; (a, b) becomes (a cos - b sin, b cos + a sin) * magnitude.  freq[i] =
     theta^(-2i/rotary_dim), stretched by `scaling` = (factor, original, fast, slow) where the spec has one: pairs
     whose wavelength is long against the original context are slowed by `factor`, short ones stay, with a linear
-    ramp over the pair index between the two (see `PositionSpec`).  The table is made once, in double precision, and
+    ramp over the pair index between the two (see `PositionSpec`); or by `wavelengths` = (factor, low, high, original),
+    which slows the pairs by where their wavelength lies.  The table is made once, in double precision, and
     rounded to float32; angle, sine and cosine are 32-bit inside the kernels that rotate.  A mixer reads `freq`,
     `rotary_dim`, `magnitude` and `pairs` and hands them to its kernel."""
 
@@ -124,6 +125,8 @@ class PairRotation:
         if rd <= 0 or rd % 2 or rd > head_dim:
             raise ValueError(f"rotary_dim {rd} must be even and at most {head_dim}")
         p = dict(spec.params)
+        if p.get("scaling") is not None and p.get("wavelengths") is not None:
+            raise ValueError("a rotation's frequencies are stretched one way or the other")
         if not spec.theta > (1.0 if p.get("scaling") is not None else 0.0):
             raise ValueError("the rotation's base must be positive, and exceed 1 where its frequencies are stretched")
         base = float(spec.theta)
@@ -135,6 +138,17 @@ class PairRotation:
             for i in range(rd // 2):
                 ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
                 freq[i] = freq[i] / factor * ramp + freq[i] * (1.0 - ramp)
+        if p.get("wavelengths") is not None:
+            factor, low, high, original = (float(v) for v in p["wavelengths"])
+            if not (factor > 0 and original > 0 and 0 < low <= high):
+                raise ValueError("wavelengths: factor, low, high and original must be positive, low at most high")
+            for i, f in enumerate(freq):
+                turns = original * f / (2.0 * math.pi)            # of this pair over the original context
+                if turns < low:
+                    freq[i] = f / factor
+                elif turns <= high:
+                    s = (turns - low) / (high - low) if high > low else 1.0
+                    freq[i] = (1.0 - s) * f / factor + s * f
         self.rotary_dim = rd
         self.magnitude = float(p.get("magnitude", 1.0))
         self.freq = torch.tensor(freq, dtype=torch.float64).to(torch.float32).to(device).contiguous()

@@ -8,7 +8,7 @@ import torch
 from ..config.specs import RejoinSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
-from .norms import PendingStart, PendingSum
+from .norms import PendingNormed, PendingStart, PendingSum
 
 
 class EmbeddingRejoin:
@@ -20,6 +20,9 @@ class EmbeddingRejoin:
     def __init__(self, spec: RejoinSpec, hidden_size: int, compute_dtype: torch.dtype):
         self.spec, self.hidden, self.dtype = spec, hidden_size, compute_dtype
         self.w_x = self.w_e = self.step = None
+
+    def matrices(self):
+        return [self.w_x, self.w_e]
 
     def parameters(self) -> Dict[str, ParamSpec]:
         return {self.spec.in_name: ParamSpec((self.hidden, 2 * self.hidden)),
@@ -47,3 +50,34 @@ class EmbeddingRejoin:
             else:
                 copy = ops.stream_norm(h, delta, None, None, None, None, 0.0, False, self.dtype, write_back=False, y2=y2)
         return PendingStart(base, self.step[t], ops.linear(copy, self.w_x, out_dtype=torch.float32, partials_ok=True))
+
+
+class AddedEmbedding:
+    """In front of every pass but the first the embedding output x0 is added to the stream.  It has no tensors: the
+    embedding kernel writes x0 twice, once as the stream, and the norm that makes the next sublayer's input adds it with
+    the output that is still pending there (`PendingNormed.join`), or, in front of a norm that does not, the stream gets it
+    in a kernel of its own."""
+
+    def __init__(self, spec: RejoinSpec, hidden_size: int, compute_dtype: torch.dtype):
+        self.spec = spec
+
+    def matrices(self):
+        return []
+
+    def parameters(self) -> Dict[str, ParamSpec]:
+        return {}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        pass
+
+    def start(self, h: torch.Tensor, delta, x0: torch.Tensor, t: int, norm):
+        """What is pending in front of `norm`, the first norm of pass t."""
+        if t == 0:
+            return delta
+        if isinstance(delta, PendingNormed) and getattr(norm, "accepts_join", False):
+            return PendingNormed(delta.y, delta.norm, join=x0)
+        ops.residual_add(h, x0)                       # a sum: what is pending may join after it
+        return delta
+
+
+REJOINS = {"linear": EmbeddingRejoin, "add": AddedEmbedding}
