@@ -17,45 +17,12 @@
 // keys 16w..16w+15 of every tile: S = Q K^T (mma.sync m16n8k16), mask, online softmax, P rounded
 // to bfloat16, O += P V.  The four warps' states are merged through shared memory at the end.
 // Built for head sizes 64 and 128 and groups up to 16; other sizes use the generic kernel.
-#include "common.cuh"
+#include "mma_tiles.cuh"
 #include <math_constants.h>
 #include <stdlib.h>
 
 #define AD_BN 64
 #define AD_THREADS 128
-
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
-    const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
-    const int bytes = valid ? 16 : 0;                 // 0: nothing is read, the 16 bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(s), "l"(gmem), "r"(bytes));
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;\n" ::); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
-__device__ __forceinline__ void ldmatrix_x4(unsigned (&r)[4], const void* smem) {
-    const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void* smem) {
-    const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const unsigned*>(&v);
-}
-// 16-byte chunk `chunk` of row `row` in a [rows][D] bfloat16 tile, XOR-swizzled against bank conflicts.
-template <int D>
-__device__ __forceinline__ bf16* tile_at(bf16* base, int row, int chunk) {
-    return base + row * D + ((chunk ^ (row & 7)) << 3);
-}
 
 // BIAS: a distance table joins the scores (an instantiation of its own, so that the plain kernel is what it was).
 template <int D, int AD_STAGES, bool BIAS>

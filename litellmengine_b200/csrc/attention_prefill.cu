@@ -13,47 +13,13 @@
 // 16-byte chunks so that ldmatrix reads are conflict-free.  Eight warps, 16 query rows each; the
 // host lists the tiles longest first (the last rows of a prompt see the most keys).
 // Built for head sizes 64 and 128; other sizes use the generic kernel.
-#include "common.cuh"
+#include "mma_tiles.cuh"
 #include <math_constants.h>
 
 #define AP_WARPS 8
 #define AP_BM (16 * AP_WARPS)      // query rows per CTA
 #define AP_BN 64                   // keys per tile
 #define AP_THREADS (32 * AP_WARPS)
-
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
-    const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
-    const int bytes = valid ? 16 : 0;                 // 0: nothing is read, the 16 bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(s), "l"(gmem), "r"(bytes));
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;\n" ::); }
-
-__device__ __forceinline__ void ldmatrix_x4(unsigned (&r)[4], const void* smem) {
-    const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void* smem) {
-    const unsigned s = static_cast<unsigned>(__cvta_generic_to_shared(smem));
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const unsigned*>(&v);
-}
-
-// Address of 16-byte chunk `chunk` of row `row` in a [rows][D] bfloat16 tile, swizzled.
-template <int D>
-__device__ __forceinline__ bf16* tile_at(bf16* base, int row, int chunk) {
-    return base + row * D + ((chunk ^ (row & 7)) << 3);
-}
 
 // EXT: the instantiation that takes a distance table, a gate per head, an output scale and an output column; the
 // plain one folds them away and is the kernel it was.

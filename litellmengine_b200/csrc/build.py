@@ -41,13 +41,14 @@ FAMILIES: Dict[str, List[str]] = {
     "attention_decode": ["attention_decode.cu"],
     "attention_prefill": ["attention_prefill.cu"],
     "attention_prefill_tcgen05": ["attention_prefill_tcgen05.cu"],
+    "attention_wide": ["attention_wide.cu"],
     "sampling": ["sampling.cu"],
     "gemm_skinny": ["gemm_skinny.cu"],
     "gemm_pair_tcgen05": ["gemm_pair_tcgen05.cu"],
     "host_core": ["host_core.cpp"],            # the host side's bookkeeping: plain C++, no device code
 }
 HOST_FAMILIES = {"host_core"}
-HEADERS = ["common.cuh", "attention_decode_noalloc.h", "attention_decode_tma.cuh"]
+HEADERS = ["common.cuh", "mma_tiles.cuh", "attention_decode_noalloc.h", "attention_decode_tma.cuh"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",

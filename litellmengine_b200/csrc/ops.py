@@ -1360,6 +1360,66 @@ def paged_attention_decode(q: torch.Tensor, out: torch.Tensor, cache: torch.Tens
     return out
 
 
+def wide_attention_supported(dk: int, dv: int, group: int) -> bool:
+    """Whether the tensor-core kernels for keys and values of any widths take this shape (`wide_attention_*`)."""
+    if dk % 8 or dv % 8:     # do not compile them just to hear "no"
+        return False
+    return bool(_fn("attention_wide", "llm_wide_attention_supported", [c_int, c_int, c_int])(dk, dv, group))
+
+
+def _wide_operands(q, out, keys, values, nq: int, nkv: int, dk: int, dv: int, page_size: int) -> None:
+    if any(t.dtype != torch.bfloat16 for t in (q, out, keys, values)):
+        raise KernelError("the attention kernels for any widths are bfloat16 only")
+    for c, w in ((keys, dk), (values, dv)):
+        if (not c.is_cuda or c.dim() != 4 or tuple(c.shape[1:]) != (nkv, page_size, w)
+                or c[0].stride() != (page_size * w, w, 1)):
+            raise KernelError("keys / values must be [pages, kv_heads, page_size, width] with dense pages")
+    if q.shape[1] != nq * dk or out.stride(1) != 1 or out.shape[0] != q.shape[0]:
+        raise KernelError("q must be [T, heads*dk] and out a matrix with T rows")
+
+
+def wide_attention_prefill(q: torch.Tensor, out: torch.Tensor, out_off: int, keys: torch.Tensor, values: torch.Tensor,
+                           tiles: torch.Tensor, n_tiles: int, entry_slot, entry_q_start, entry_q_len, entry_kv_len,
+                           block_table: torch.Tensor, nq: int, nkv: int, dk: int, dv: int, page_size: int,
+                           window: Optional[int], scale: float, status: torch.Tensor, out_scale: float = 1.0) -> None:
+    """`paged_attention_prefill` for keys of width dk and values of width dv (multiples of 8 up to 256) in tensors of their
+    own; the result times `out_scale` goes to columns out_off .. out_off + nq*dv of `out`.  bfloat16 only."""
+    _dev(q, tiles, entry_slot, entry_q_start, entry_q_len, entry_kv_len, block_table, status)
+    _wide_operands(q, out, keys, values, nq, nkv, dk, dv, page_size)
+    f = _fn("attention_wide", "llm_wide_attention_prefill",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_float, c_longlong, c_int, c_void_p])
+    _check(f(_ptr(q), _ptr(out), _ptr(keys), _ptr(values), keys.stride(0), values.stride(0), _ptr(tiles), n_tiles, _ptr(entry_slot),
+             _ptr(entry_q_start), _ptr(entry_q_len), _ptr(entry_kv_len), _ptr(block_table), block_table.shape[1], nq, nkv, dk, dv,
+             page_size, int(window) if window else 0, float(scale), keys.shape[0], _ptr(status), float(out_scale), out.stride(0),
+             out_off, _stream()), "wide_attention_prefill")
+
+
+def wide_attention_decode(q: torch.Tensor, out: torch.Tensor, out_off: int, keys: torch.Tensor, values: torch.Tensor,
+                          rows: Optional[torch.Tensor], n_rows: int, positions, token_entry, entry_slot,
+                          block_table: torch.Tensor, nq: int, nkv: int, dk: int, dv: int, page_size: int,
+                          window: Optional[int], scale: float, num_splits: int, status: torch.Tensor,
+                          out_scale: float = 1.0) -> None:
+    """`paged_attention_decode` (single decoded tokens, the keys split `num_splits` ways) for keys and values of widths of
+    their own, as in `wide_attention_prefill`."""
+    _dev(q, rows, positions, token_entry, entry_slot, block_table, status)
+    _wide_operands(q, out, keys, values, nq, nkv, dk, dv, page_size)
+    need = _fn("attention_wide", "llm_wide_decode_scratch_floats", [c_int, c_int, c_int, c_int],
+               restype=c_longlong)(n_rows, nq, dv, num_splits)
+    scratch = decode_scratch(q.device, int(need))
+    f = _fn("attention_wide", "llm_wide_attention_decode",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float, c_longlong, c_int,
+             c_void_p])
+    _check(f(_ptr(q), _ptr(out), _ptr(keys), _ptr(values), keys.stride(0), values.stride(0), _ptr(rows), n_rows, _ptr(positions),
+             _ptr(token_entry), _ptr(entry_slot), _ptr(block_table), block_table.shape[1], nq, nkv, dk, dv, page_size,
+             int(window) if window else 0, float(scale), keys.shape[0], num_splits, _ptr(scratch), _ptr(status), float(out_scale),
+             out.stride(0), out_off, _stream()), "wide_attention_decode")
+    if num_splits > 1:
+        global launch_count
+        launch_count += 1                         # the merge kernel
+
+
 def paged_attention_prefill(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, tiles: torch.Tensor,
                             n_tiles: int, entry_slot, entry_q_start, entry_q_len, entry_kv_len,
                             block_table: torch.Tensor, nq: int, nkv: int, d: int, page_size: int,

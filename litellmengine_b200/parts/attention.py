@@ -302,6 +302,10 @@ class GatedAttentionMixer(BranchMixer):
                               and self.device.type == "cuda" and (self.gate_per_head or not spec.output_gate)
                               and ops.prefill_attention_supported(self.d))
         self._tuned_decode = self._tuned_prompt and ops.fast_attention_supported(self.d, self.nq // self.nkv)
+        # any other widths, plain scores over a plain walk: the tensor-core kernels that take keys and values as they are
+        self._wide = (not self._tuned and not self._tuned_prompt and compute_dtype == torch.bfloat16 and self.device.type == "cuda"
+                      and spec.distance_bias is None and not scored and not walked
+                      and ops.wide_attention_supported(self.d, self.dv, self.nq // self.nkv))
         self.dist_table_t = None
         self.analytic = False                   # dist_table_t holds (temperature, r1, r2) per head instead of a table
 
@@ -373,7 +377,7 @@ class GatedAttentionMixer(BranchMixer):
                          self.spec.chunk)
 
     def step_prelude(self):
-        return AttentionWork() if self._tuned or self._tuned_prompt else None
+        return AttentionWork() if self._tuned or self._tuned_prompt or self._wide else None
 
     @property
     def graph_variant_group(self):
@@ -382,12 +386,12 @@ class GatedAttentionMixer(BranchMixer):
     def graph_variant(self, batch, padded: bool) -> int:
         if self._tuned:
             return AttentionMixer.graph_variant(self, batch, padded)
-        if not self._tuned_decode:
+        if not self._tuned_decode and not self._wide:
             return 0
         work = batch.preludes.get(AttentionWork.name)       # the decode kernel's key splits, as the step will choose them
         n_dec = 0 if work is None else (work.padded_rows.shape[0] if padded else work.num_decode)
         n_tiles = 0 if work is None else (work.padded_tiles.shape[0] if padded else work.num_prefill_tiles)
-        return decode_key_splits(self.device, n_dec, self.nkv, decode_reach(batch, self.span)) if n_dec and not n_tiles else 0
+        return decode_key_splits(self.device, n_dec, self.nkv, decode_reach(batch, self.span)) if n_dec and (self._wide or not n_tiles) else 0
 
     def mix(self, proj, col0, ctx, out, out_col0, out_scale):
         b, s = ctx.batch, self.spec
@@ -406,6 +410,9 @@ class GatedAttentionMixer(BranchMixer):
             a = attention_over_pages(q, ctx, self.nq, self.nkv, self.d, self.span, self.scale, out=out if direct else None)
             if not direct:
                 ops.gate_mul(a, proj, col0 + self.g_off, out, out_col0, s.output_gate, out_scale)
+            return
+        if self._wide and b.preludes.get(AttentionWork.name) is not None:
+            self._mix_wide(q, proj, col0, ctx, out, out_col0, out_scale)
             return
         work = b.preludes.get(AttentionWork.name) if self._tuned_prompt and ctx.cache is not None else None
         padded = getattr(b, "any_division", False)
@@ -457,6 +464,30 @@ class GatedAttentionMixer(BranchMixer):
             dist_bias=self.dist_table, gate_per_head=self.gate_per_head, rows=rows, head_scale=self.head_temp,
             log_bias=(self.log_r1, self.log_r2) if self.log_r1 is not None else None, keep_first=self.keep_first,
             sink=self.sink)
+
+
+    def _mix_wide(self, q, proj, col0, ctx, out, out_col0, out_scale):
+        """Prompt portions and single tokens in the tensor-core kernels for keys and values of any widths; a gate in a small
+        kernel after them."""
+        b, s = ctx.batch, self.spec
+        work, padded = b.preludes[AttentionWork.name], getattr(b, "any_division", False)
+        n_dec = work.padded_rows.shape[0] if padded else work.num_decode
+        n_tiles = work.padded_tiles.shape[0] if padded else work.num_prefill_tiles
+        a, at, by = (out, out_col0, out_scale) if not s.output_gate else (
+            torch.empty((q.shape[0], self.out_width), dtype=self.dtype, device=q.device), 0, 1.0)
+        shape = (ctx.block_table, self.nq, self.nkv, self.d, self.dv, ctx.page_size, self.span, self.scale)
+        if n_dec:
+            rows = work.padded_rows if padded else (None if n_dec == b.num_tokens else work.decode_rows)
+            splits = decode_key_splits(q.device, n_dec, self.nkv, decode_reach(b, self.span))
+            ops.wide_attention_decode(q, a, at, ctx.cache_keys, ctx.cache_values, rows, n_dec, b.positions, b.token_entry,
+                                      b.entry_slot, *shape, splits, ctx.status, out_scale=by)
+        if n_tiles:
+            ops.wide_attention_prefill(q, a, at, ctx.cache_keys, ctx.cache_values, work.padded_tiles if padded else work.prefill_tiles,
+                                       n_tiles, b.entry_slot, b.entry_q_start, b.entry_q_len, b.entry_kv_len, *shape, ctx.status,
+                                       out_scale=by)
+        if s.output_gate:
+            ops.gate_mul(a, proj, col0 + self.g_off, out, out_col0, s.output_gate, out_scale,
+                         per_head=self.dv if self.gate_per_head else 0)
 
 
 def distance_bucket(n: int, rows: int, far: float) -> int:
