@@ -2,7 +2,7 @@
 """Benchmark of the engine on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers L]
-                    [--impl ours|reference] [--points LIST | --no-points] [--design tobovik|gubidra|komazen|vugedra|pukatar [--sizes LIST]]
+                    [--impl ours|reference] [--points LIST | --no-points] [--design tobovik|gubidra|komazen|vugedra|pukatar|purivik [--sizes LIST]]
 
 Headline (`value`): decode tokens/s of `batch` requests whose context ends at 4,096 tokens, on a
 model with the layer sizes of Qwen3-8B (36 layers unless --layers says fewer; the JSON names both
@@ -22,7 +22,7 @@ prefill and decode of the Tobovik design beside Qwen3 at equal width, heads, fee
 vocabulary, and the design's own kernels beside the like kernels of the Qwen3 path with their roofline
 fractions.  `--design gubidra` does the same for the Gubidra design beside Tobovik, its closest model, and
 `--design komazen` for the Komazen design beside Qwen3, `--design vugedra` for the Vugedra design beside Gubidra,
-`--design pukatar` for the Pukatar design beside Vugedra.
+`--design pukatar` for the Pukatar design beside Vugedra, `--design purivik` for the Purivik design beside Vugedra.
 Without it the workload and the line above are what they always were.
 
 `--impl reference` times the unmodified reference engine (float32, its only precision) on the same
@@ -931,6 +931,164 @@ def pukatar_bench(args, pk, measure) -> int:
     return 0
 
 
+def purivik_dict(width, ff, heads, kv, layers, vdim=None):
+    """Attention within chunks of 1,024 positions in every layer (keys of 128, a rotation of half a head with frequencies
+    stretched by wavelength), a clamped dense feed-forward and eight experts of half its size (two chosen, the weight on
+    their input) in turns; the second half of the layers is a loop of one pass, so that the embedding is kept for it."""
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2}}
+    mixer = {"heads": heads, "kv_heads": kv, "dim": DESIGN_HEAD, "vdim": vdim or DESIGN_HEAD, "scale": DESIGN_HEAD ** -0.5, "mask": {"size": 1024},
+             "rot": {"base": 10000.0, "dims": DESIGN_HEAD // 2, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 1024}}}
+    return {"architecture": "Purivik", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": 4.0}, "norm": {"eps": 1e-5},
+            "residual_mult": 0.5, "loop": {"start": layers // 2, "stop": layers, "times": 1},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": (dense, moe)[i % 2]} for i in range(layers)]}
+
+
+def vugedra_attention_dict(width, ff, heads, kv, layers, vdim=None):
+    """Vugedra with attention in every layer (a window of 1,024 without kept keys) and the feed-forwards of `purivik_dict`:
+    no shared expert, no outputs that are no experts."""
+    cfg = vugedra_dict(width, ff, heads, kv, layers)
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2}}
+    mixer = dict(cfg["layers"][0]["mixer"], vdim=vdim or DESIGN_HEAD, mask={"size": 1024})
+    return dict(cfg, layers=[{"type": "attention", "mixer": mixer, "mlp": (dense, moe)[i % 2]} for i in range(layers)])
+
+
+def purivik_bench(args, pk, measure) -> int:
+    """`--design purivik`: the design beside Vugedra (the closest model: norms on both sides of every sublayer, attention over
+    the last keys, routed experts), both with attention in every layer, at equal width, heads, feed-forwards, depth and
+    vocabulary, with values as wide as the keys and with wider ones; and its kernels beside their like."""
+    import torch
+    from litellmengine_b200.config import config_from_dict
+    from litellmengine_b200.csrc import ops
+    from litellmengine_b200.csrc.microbench import Flusher, timed
+    dev = "cuda:0"
+    sizes = {}
+    for name, (width, ff, heads, kv, layers) in DESIGN_SIZES.items():
+        if args.sizes and name not in args.sizes.split(","):
+            continue
+        for tag, vdim in (("", None), ("_values_192", 192)):
+            rec = sizes[name + tag] = {"shape": {"width": width, "ff": ff, "heads": heads, "kv_heads": kv, "layers": layers, "vocab": DESIGN_VOCAB,
+                                                 "key_width": DESIGN_HEAD, "value_width": vdim or DESIGN_HEAD}}
+            for label, cfg in (("purivik", purivik_dict(width, ff, heads, kv, layers, vdim)),
+                               ("vugedra", vugedra_attention_dict(width, ff, heads, kv, layers, vdim))):
+                rec[label] = measure(config_from_dict(cfg))
+                gc.collect()
+                torch.cuda.empty_cache()
+            rec["purivik_over_vugedra"] = {k: round(rec["purivik"][k] / rec["vugedra"][k], 3) for k in rec["purivik"] if k.endswith("tok_s")}
+    flush = Flusher(dev)
+    width, ff, heads, kv, _ = DESIGN_SIZES["w4096"]
+    T, hbm, d = 2048, pk["hbm_gbs"] * 1e9, DESIGN_HEAD
+    tensor_peak = pk.get("bf16_tflops", 1590.0) * 1e12
+    kernels = {}
+
+    def add(name, fn, nbytes=None, flops=None):
+        sec = timed(fn, 10, 3, flush)
+        rec = {"us": round(sec * 1e6, 2)}
+        if nbytes is not None:
+            rec.update(gbs=round(nbytes / sec / 1e9, 1), frac_of_hbm=round(nbytes / sec / hbm, 4))
+        if flops is not None:
+            rec.update(tflops=round(flops / sec / 1e12, 2), frac_of_bf16_peak=round(flops / sec / tensor_peak, 4))
+        kernels[name] = rec
+
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32, device=dev)
+    bf = lambda *s: torch.randn(*s, device=dev).to(torch.bfloat16)
+    status = torch.zeros(2, dtype=torch.int32, device=dev)
+    # between the sublayers; the embedding
+    for n in (T, 8):
+        h, y, x0 = (torch.randn(n, width, device=dev) for _ in range(3))
+        w, row, one = torch.ones(width, device=dev), torch.zeros(width, device=dev), torch.ones(1, device=dev)
+        nb = n * width * (4 + 4 + 4 + 2)
+        add(f"rmsnorm_sandwich (new): {n} tokens", lambda: ops.rmsnorm_sandwich(h, y, (w, 1e-5), (w, 1e-5), torch.bfloat16), nbytes=nb)
+        add(f"rmsnorm_sandwich, the embedding joins (new): {n} tokens",
+            lambda: ops.rmsnorm_sandwich(h, y, (w, 1e-5), (w, 1e-5), torch.bfloat16, join=x0), nbytes=nb + n * width * 4)
+        add(f"tanh_norm (like: Vugedra's norm around the residual add): {n} tokens",
+            lambda: ops.tanh_norm(h, y, (one, w, row), (one, w, row), torch.bfloat16), nbytes=nb)
+        add(f"rmsnorm with the residual add (like: one norm): {n} tokens", lambda: ops.rmsnorm(h, w, 1e-5, torch.bfloat16, delta=y, write_sum=True), nbytes=nb)
+    h, x0 = (torch.empty(T, width, device=dev) for _ in range(2))
+    table, ids = bf(DESIGN_VOCAB, width), torch.randint(0, DESIGN_VOCAB, (T,), device=dev, dtype=torch.int32)
+    add("embedding, written twice (new)", lambda: ops.embedding(ids, table, status, scale=4.0, out=h, keep=x0), nbytes=T * width * (2 + 4 + 4))
+    add("embedding (like)", lambda: ops.embedding(ids, table, status, scale=4.0, out=h), nbytes=T * width * (2 + 4))
+    # attention
+    pages = T // PAGE
+    cache, tbl = bf(pages, 2, kv, PAGE, d), torch.arange(pages, device=dev, dtype=torch.int32).view(1, pages)
+    qa = bf(T, heads * d)
+    oa = torch.empty_like(qa)
+    tiles = i32([(0, r0) for r0 in range(0, T, ops.PREFILL_TILE_ROWS)][::-1])
+    e0, e_len, sinks = i32([0]), i32([T]), torch.zeros(heads, device=dev)
+    entry = (tiles, tiles.shape[0], e0, e0, e_len, e_len, tbl, heads, kv)
+    chunk = 1024
+    seen = {-chunk: sum(p % chunk + 1 for p in range(T)), chunk: sum(min(p + 1, chunk) for p in range(T)), None: T * (T + 1) // 2}
+    flops = lambda span, dk, dv: 2.0 * heads * (dk + dv) * seen[span]
+    for label, span in ((f"chunks of {chunk} (new)", -chunk), (f"a window of {chunk} (like)", chunk), ("all keys (like)", None)):
+        add(f"prompt attention, tcgen05, {label}: {T} tokens", lambda span=span: ops.paged_attention_prefill_tcgen05(qa, oa, cache, *entry, d, PAGE, span, d ** -0.5, status),
+            flops=flops(span, d, d))
+    add(f"prompt attention, mma, a window of {chunk} with a sink and kept keys (like: Vugedra's): {T} tokens",
+        lambda: ops.paged_attention_prefill_biased(qa, oa, 0, cache, *entry, d, PAGE, chunk, d ** -0.5, status, keep_first=4, sink=sinks), flops=flops(chunk, d, d))
+    for dk, dv in ((64, 80), (128, 192), (128, 128), (256, 256)):
+        keys, values = bf(pages, kv, PAGE, dk), bf(pages, kv, PAGE, dv)
+        q, o = bf(T, heads * dk), torch.empty(T, heads * dv, device=dev, dtype=torch.bfloat16)
+        add(f"prompt attention, keys of {dk}, values of {dv}, chunks of {chunk} (new): {T} tokens",
+            lambda: ops.wide_attention_prefill(q, o, 0, keys, values, *entry, dk, dv, PAGE, -chunk, dk ** -0.5, status), flops=flops(-chunk, dk, dv))
+        if (dk, dv) == (128, 192):
+            pos, zero = torch.arange(T, device=dev, dtype=torch.int32), torch.zeros(T, device=dev, dtype=torch.int32)
+            add(f"prompt attention, keys of {dk}, values of {dv}, a window of {chunk}, general kernel (like: Vugedra's): {T} tokens",
+                lambda: ops.paged_attention_generic_kv(q, keys, values, pos, zero, e0, tbl, heads, kv, dk, dv, PAGE, chunk, dk ** -0.5, status, o),
+                flops=flops(chunk, dk, dv))
+    Bd, ctx = 64, 2048
+    dpages = ctx // PAGE
+    dtbl = torch.arange(Bd * dpages, device=dev, dtype=torch.int32).view(Bd, dpages)
+    dpos, dent = torch.full((Bd,), ctx - 1, device=dev, dtype=torch.int32), torch.arange(Bd, device=dev, dtype=torch.int32)
+    step = (None, Bd, dpos, dent, dent, dtbl, heads, kv)
+    dcache = bf(Bd * dpages, 2, kv, PAGE, d)
+    kv_bytes = lambda dk, dv: Bd * chunk * kv * (dk + dv) * 2
+    for label, span in ((f"a chunk of {chunk} (new)", -chunk), (f"a window of {chunk} (like)", chunk)):
+        add(f"decode attention, {label}: {Bd} tokens at position {ctx - 1}",
+            lambda span=span: ops.paged_attention_decode(qa[:Bd], oa[:Bd], dcache, *step, d, PAGE, span, d ** -0.5, 1, status), nbytes=kv_bytes(d, d))
+    del dcache
+    for dk, dv in ((64, 80), (128, 192), (128, 128)):
+        keys, values = bf(Bd * dpages, kv, PAGE, dk), bf(Bd * dpages, kv, PAGE, dv)
+        q, o = bf(Bd, heads * dk), torch.empty(Bd, heads * dv, device=dev, dtype=torch.bfloat16)
+        for splits in (1, 2):
+            add(f"decode attention, keys of {dk}, values of {dv}, a chunk of {chunk}, {splits} splits (new): {Bd} tokens at position {ctx - 1}",
+                lambda: ops.wide_attention_decode(q, o, 0, keys, values, *step, dk, dv, PAGE, -chunk, dk ** -0.5, splits, status), nbytes=kv_bytes(dk, dv))
+        if (dk, dv) == (128, 192):
+            add(f"decode attention, keys of {dk}, values of {dv}, a window of {chunk}, general kernel (like: Vugedra's): {Bd} tokens",
+                lambda: ops.paged_attention_generic_kv(q, keys, values, dpos, dent, dent, dtbl, heads, kv, dk, dv, PAGE, chunk, dk ** -0.5, status, o),
+                nbytes=kv_bytes(dk, dv))
+    # the feed-forwards
+    x, wgu = bf(T, width), bf(2 * ff, width)
+    act = torch.empty(T, ff, device=dev, dtype=torch.bfloat16)
+    for label, kind in (("clamped (new)", "clamped_swish"), ("silu (like)", "silu")):
+        add(f"paired product with the activation in its epilogue, {label}: {T} x {2 * ff} x {width}",
+            lambda kind=kind: ops.linear_pair_silu_mul(x, wgu, out=act, activation=kind, limit=7.0), flops=4.0 * T * ff * width)
+    gu = bf(T, 2 * ff)
+    for label, kind in (("clamped (new)", "clamped_swish"), ("silu (like)", "silu")):
+        add(f"activation alone, {label}: {T} x {ff}", lambda kind=kind: ops.silu_and_mul(gu, out=act, activation=kind, limit=7.0), nbytes=T * ff * 6)
+    E, top, fe = 8, 2, ff // 2
+    wr = torch.randn(E, width, device=dev) * width ** -0.5
+    route_bytes = T * (width * 2 + E * 4)
+    add("moe_route, sigmoid scores as they are (new)", lambda: ops.moe_route(x, wr, top, None, 1.0, normalize=False), nbytes=route_bytes)
+    add("moe_route, sigmoid with groups, shares of one (like)", lambda: ops.moe_route(x, wr, top, (4, 2), 1.0), nbytes=route_bytes)
+    dense, eids, wts = ops.moe_route(x, wr, top, None, 1.0, normalize=False, lists=True)
+    w1, w2 = bf(E * 2 * fe, width), bf(width, E * fe)
+    inf = float("inf")
+    for label, on in (("weight on the input (new)", True), ("weight on the output (like)", False)):
+        add(f"routed experts, sorted tokens, {label}: {T} tokens (8 kernels, two grouped products)",
+            lambda on=on: ops.moe_sorted(x, w1, w2, eids, wts, E, fe, inf, 1.0, shift=0.0, on_input=on), flops=6.0 * T * top * fe * width)
+        add(f"routed experts, chosen matrices only, {label}: 2 tokens", lambda on=on: ops.moe_sparse(x[:2], w1, w2, eids[:2], wts[:2], fe, inf, 1.0, shift=0.0, on_input=on),
+            nbytes=float(len(set(eids[:2].flatten().tolist()))) * 3 * fe * width * 2)
+        gue = torch.randn(64, E * 2 * fe, device=dev)
+        add(f"moe_act, {label}: 64 tokens", lambda on=on: ops.moe_act(gue, dense[:64].contiguous(), E, fe, inf, 1.0, torch.bfloat16, shift=0.0, on_input=on),
+            nbytes=64 * (top * 2 * fe * 4 + E * fe * 2))
+    print(json.dumps({"metric": "tokens/s of the Purivik design beside Vugedra at equal sizes (bfloat16, random weights)",
+                      "design": "purivik", "prompt_tokens": 2048, "decode_context": 1024, "steps": args.steps,
+                      "warmup": args.warmup, "sizes": sizes, "kernels_at_w4096": kernels,
+                      "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": round(tensor_peak / 1e12, 1), "source": pk["source"]},
+                      "l2": "kernel timings: a 256 MB buffer is overwritten between launches; steps read every weight"}))
+    return 0
+
+
 def komazen_bench(args, pk, measure) -> int:
     """`--design komazen`: the design beside Qwen3 (the closest model: softmax attention and a dense gated feed-forward
     in every layer) at equal width, heads, feed-forward, depth and vocabulary, and its kernels beside their like."""
@@ -1324,6 +1482,8 @@ def design_bench(args, pk) -> int:
         return vugedra_bench(args, pk, measure)
     if args.design == "pukatar":
         return pukatar_bench(args, pk, measure)
+    if args.design == "purivik":
+        return purivik_bench(args, pk, measure)
     sizes = {}
     for name, (width, ff, heads, kv, layers) in DESIGN_SIZES.items():
         if args.sizes and name not in args.sizes.split(","):
@@ -1443,9 +1603,9 @@ def main() -> int:
     ap.add_argument("--points", default=",".join(ALL_POINTS),
                     help="which extra measurements to take: " + ",".join(ALL_POINTS))
     ap.add_argument("--no-points", action="store_true", help="the headline, prefill and e2e only")
-    ap.add_argument("--design", choices=["tobovik", "gubidra", "komazen", "vugedra", "pukatar"],
+    ap.add_argument("--design", choices=["tobovik", "gubidra", "komazen", "vugedra", "pukatar", "purivik"],
                     help="instead of the default workload: this design beside its closest model (tobovik and komazen beside "
-                         "Qwen3, gubidra beside tobovik, vugedra beside gubidra, pukatar beside vugedra) at equal sizes, and its kernels")
+                         "Qwen3, gubidra beside tobovik, vugedra beside gubidra, pukatar and purivik beside vugedra) at equal sizes, and its kernels")
     ap.add_argument("--sizes", default="", help="with --design: which of " + ",".join(DESIGN_SIZES) + " (default: all)")
     args = ap.parse_args()
 

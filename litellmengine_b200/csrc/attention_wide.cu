@@ -8,12 +8,13 @@
 //                         two in shared memory.
 //   wide_decode_kernel    single tokens, split over the keys: a CTA takes one token, one kv head and one of the splits;
 //                         the group's query heads are the 16 rows of its products, its 4 warps take 16 keys each of
-//                         every tile, three tiles in shared memory.  Partial results are merged by
+//                         every tile, two tiles in shared memory (so that two CTAs or more share an SM: a warp's
+//                         work on its 16 keys is a chain of latencies).  Partial results are merged by
 //                         wide_combine_kernel (maxima in the base-2 domain).
 // The formulas are those of the kernels for head sizes 64 and 128 (`attention_prefill.cu`, `attention_decode.cu`); what
 // differs is that rows of dk and dv entries lie in shared memory at a stride of one chunk more than they are long (an
-// odd number of sixteen-byte chunks, so that eight rows fall into different banks) and that the accumulators' width is a
-// compile-time bound DV with blocks past dv skipped.
+// odd number of sixteen-byte chunks, so that eight rows fall into different banks) and that value rows are padded with
+// zeros to a compile-time width DV, so that the products with them have no conditions in them.
 #include "mma_tiles.cuh"
 #include <math_constants.h>
 
@@ -23,10 +24,10 @@
 #define WP_THREADS (32 * WP_WARPS)
 #define WD_BN 64
 #define WD_THREADS 128
-#define WD_STAGES 3
 
 static __host__ __device__ __forceinline__ int wide_pad(int d) { return (d + 15) / 16 * 16; }        // entries computed
 static __host__ __device__ __forceinline__ int wide_row(int d) { return wide_pad(d) + 8; }           // entries from row to row
+static int wide_dv(int dv) { return dv <= 64 ? 64 : dv <= 96 ? 96 : dv <= 128 ? 128 : dv <= 160 ? 160 : dv <= 192 ? 192 : 256; }
 
 // Where a key's row and a value's row lie, found once per key.
 struct WideCache {
@@ -37,7 +38,7 @@ struct WideCache {
 };
 
 template <int DV>
-__global__ void __launch_bounds__(WP_THREADS) wide_prefill_kernel(
+__global__ void __launch_bounds__(WP_THREADS, DV <= 96 ? 2 : 1) wide_prefill_kernel(
     const bf16* __restrict__ q, bf16* __restrict__ out, const WideCache c, const int32_t* __restrict__ tiles,
     const int32_t* __restrict__ entry_slot, const int32_t* __restrict__ entry_q_start,
     const int32_t* __restrict__ entry_q_len, const int32_t* __restrict__ entry_kv_len,
@@ -45,7 +46,8 @@ __global__ void __launch_bounds__(WP_THREADS) wide_prefill_kernel(
     int32_t* __restrict__ status, float out_scale, long long out_stride, int out_off) {
     pdl_begin();
     extern __shared__ __align__(128) unsigned char smem_raw[];
-    const int dk16 = wide_pad(c.dk), dv16 = wide_pad(c.dv), ldk = wide_row(c.dk), ldv = wide_row(c.dv);
+    constexpr int ldv = DV + 8;
+    const int dk16 = wide_pad(c.dk), ldk = wide_row(c.dk);
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                    // [BM][ldk]
     bf16* k_s = q_s + WP_BM * ldk;                                    // [2][64][ldk]
     bf16* v_s = k_s + 2 * WP_BN * ldk;                                // [2][64][ldv]
@@ -84,7 +86,7 @@ __global__ void __launch_bounds__(WP_THREADS) wide_prefill_kernel(
         bf16* kd = k_s + (buf * WP_BN + ld_row) * ldk;
         bf16* vd = v_s + (buf * WP_BN + ld_row) * ldv;
         for (int ch = ld_sub * 8; ch < dk16; ch += TPR * 8) cp_async16(kd + ch, ch < c.dk ? ks + ch : ks, valid && ch < c.dk);
-        for (int ch = ld_sub * 8; ch < dv16; ch += TPR * 8) cp_async16(vd + ch, ch < c.dv ? vs + ch : vs, valid && ch < c.dv);
+        for (int ch = ld_sub * 8; ch < DV; ch += TPR * 8) cp_async16(vd + ch, ch < c.dv ? vs + ch : vs, valid && ch < c.dv);
     };
     {
         constexpr int TPQ = WP_THREADS / WP_BM;
@@ -179,7 +181,6 @@ __global__ void __launch_bounds__(WP_THREADS) wide_prefill_kernel(
         const bf16* va = vd + ((lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8;
 #pragma unroll
         for (int np = 0; np < DV / 16; ++np) {
-            if (np * 16 >= dv16) break;
             o[2 * np][0] *= al0; o[2 * np][1] *= al0; o[2 * np][2] *= al1; o[2 * np][3] *= al1;
             o[2 * np + 1][0] *= al0; o[2 * np + 1][1] *= al0; o[2 * np + 1][2] *= al1; o[2 * np + 1][3] *= al1;
             unsigned vf[WP_BN / 16][4];
@@ -216,10 +217,11 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
     float out_scale, long long out_stride, int out_off) {
     pdl_begin();
     extern __shared__ __align__(128) unsigned char smem_raw[];
-    const int dk16 = wide_pad(c.dk), dv16 = wide_pad(c.dv), ldk = wide_row(c.dk), ldv = wide_row(c.dv);
+    constexpr int ldv = DV + 8;
+    const int dk16 = wide_pad(c.dk), ldk = wide_row(c.dk);
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);                 // [16][ldk]
-    bf16* k_s = q_s + 16 * ldk;                                    // [STAGES][64][ldk]
-    bf16* v_s = k_s + WD_STAGES * WD_BN * ldk;                     // [STAGES][64][ldv]
+    bf16* k_s = q_s + 16 * ldk;                                    // [2][64][ldk]
+    bf16* v_s = k_s + 2 * WD_BN * ldk;                             // [2][64][ldv]
     __shared__ float m_s[4][16], l_s[4][16];
 
     const int split = blockIdx.x, kvh = blockIdx.y, r = blockIdx.z;
@@ -260,7 +262,7 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
 #pragma unroll 4
         for (int ch = ld_half * 8; ch < dk16; ch += 16) cp_async16(kd + ch, ch < c.dk ? ks + ch : ks, valid && ch < c.dk);
 #pragma unroll 4
-        for (int ch = ld_half * 8; ch < dv16; ch += 16) cp_async16(vd + ch, ch < c.dv ? vs + ch : vs, valid && ch < c.dv);
+        for (int ch = ld_half * 8; ch < DV; ch += 16) cp_async16(vd + ch, ch < c.dv ? vs + ch : vs, valid && ch < c.dv);
     };
 
     if (n_tiles > 0) {
@@ -272,12 +274,7 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
         load_kv(k_begin, 0, lookup(k_begin));
     }
     cp_async_commit();
-#pragma unroll
-    for (int st = 1; st < WD_STAGES - 1; ++st) {
-        if (st < n_tiles) load_kv(k_begin + st * WD_BN, st, lookup(k_begin + st * WD_BN));
-        cp_async_commit();
-    }
-    int page_ahead = (WD_STAGES - 1 < n_tiles) ? lookup(k_begin + (WD_STAGES - 1) * WD_BN) : -2;
+    int page_ahead = n_tiles > 1 ? lookup(k_begin + WD_BN) : -2;
 
     float o[DV / 8][4];
 #pragma unroll
@@ -286,24 +283,37 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
     const bf16* qa = q_s + ((lane & 7) + ((lane >> 3) & 1) * 8) * ldk + (lane >> 4) * 8;
 
     for (int it = 0; it < n_tiles; ++it) {
-        const int kt = k_begin + it * WD_BN, buf = it % WD_STAGES;
-        cp_async_wait<WD_STAGES - 2>();                             // tile `it` has landed; later ones may be in flight
-        __syncthreads();                                            // and every warp is done with tile it-1's buffer
-        if (it + WD_STAGES - 1 < n_tiles) load_kv(kt + (WD_STAGES - 1) * WD_BN, (it + WD_STAGES - 1) % WD_STAGES, page_ahead);
+        const int kt = k_begin + it * WD_BN, buf = it & 1;
+        cp_async_wait_all();
+        __syncthreads();                                            // tile `it` has landed, and every warp is done with tile it-1's buffer
+        if (it + 1 < n_tiles) load_kv(kt + WD_BN, buf ^ 1, page_ahead);
         cp_async_commit();
-        page_ahead = (it + WD_STAGES < n_tiles) ? lookup(kt + WD_STAGES * WD_BN) : -2;
+        page_ahead = it + 2 < n_tiles ? lookup(kt + 2 * WD_BN) : -2;
         const int key0 = kt + warp * 16;                            // this warp's 16 keys of the tile
         if (key0 >= k_end) continue;                                // warp-uniform: nothing of ours in this tile
         const bf16* ka = k_s + (buf * WD_BN + warp * 16 + (lane & 7) + (lane >> 4) * 8) * ldk + ((lane >> 3) & 1) * 8;
-        float s[2][4];
-        s[0][0] = s[0][1] = s[0][2] = s[0][3] = s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.0f;
-#pragma unroll 4
-        for (int kb = 0; kb < dk16; kb += 16) {
+        float s[2][4], s2[2][4];                                    // even and odd blocks of 16 key entries: two chains
+#pragma unroll
+        for (int u = 0; u < 4; ++u) s[0][u] = s[1][u] = s2[0][u] = s2[1][u] = 0.0f;
+#pragma unroll 2
+        for (int kb = 0; kb < dk16; kb += 32) {
             unsigned qf[4], b[4];
             ldmatrix_x4(qf, qa + kb);
             ldmatrix_x4(b, ka + kb);
             mma_bf16(s[0], qf, b[0], b[1]);
             mma_bf16(s[1], qf, b[2], b[3]);
+            if (kb + 16 < dk16) {
+                unsigned qf2[4], b2[4];
+                ldmatrix_x4(qf2, qa + kb + 16);
+                ldmatrix_x4(b2, ka + kb + 16);
+                mma_bf16(s2[0], qf2, b2[0], b2[1]);
+                mma_bf16(s2[1], qf2, b2[2], b2[3]);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            s[0][u] += s2[0][u];
+            s[1][u] += s2[1][u];
         }
         float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
@@ -338,7 +348,6 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
         const bf16* va = v_s + (buf * WD_BN + warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8;
 #pragma unroll
         for (int np = 0; np < DV / 16; ++np) {
-            if (np * 16 >= dv16) break;
             unsigned b[4];
             ldmatrix_x4_trans(b, va + np * 16);
             o[2 * np][0] *= al0; o[2 * np][1] *= al0; o[2 * np][2] *= al1; o[2 * np][3] *= al1;
@@ -350,7 +359,7 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
     cp_async_wait_all();
     __syncthreads();                                                // tiles are done: reuse their memory
 
-    const int as = dv16 + 8;                                        // row stride: rows 0..3 hit different banks
+    constexpr int as = DV + 8;                                      // row stride: rows 0..3 hit different banks
     float* acc_s = reinterpret_cast<float*>(k_s);                   // [4 warps][16 rows][as]; only rows < G are used
     {
         const int r0 = lane >> 2;
@@ -358,7 +367,6 @@ __global__ void __launch_bounds__(WD_THREADS) wide_decode_kernel(
         float* a1 = a0 + 8 * as;
 #pragma unroll
         for (int nb = 0; nb < DV / 8; ++nb) {
-            if (nb * 8 >= dv16) break;
             if (r0 < G) *reinterpret_cast<float2*>(a0 + nb * 8) = make_float2(o[nb][0], o[nb][1]);
             if (r0 + 8 < G) *reinterpret_cast<float2*>(a1 + nb * 8) = make_float2(o[nb][2], o[nb][3]);
         }
@@ -431,10 +439,14 @@ static int wide_check(const void* q, const void* keys, const void* values, long 
 }
 
 #define WIDE_BY_DV(LAUNCH)       \
-    if (dv <= 64) LAUNCH(64);    \
-    else if (dv <= 128) LAUNCH(128); \
-    else if (dv <= 192) LAUNCH(192); \
-    else LAUNCH(256)
+    switch (wide_dv(dv)) {       \
+        case 64: LAUNCH(64); break;   \
+        case 96: LAUNCH(96); break;   \
+        case 128: LAUNCH(128); break; \
+        case 160: LAUNCH(160); break; \
+        case 192: LAUNCH(192); break; \
+        default: LAUNCH(256);    \
+    }
 
 // q: bfloat16 [T, nq*dk]; keys / values: bfloat16 [pages, nkv, page_size, dk / dv], `key_page` / `value_page` elements from
 // page to page; tiles: int32 [n_tiles][2] = (entry, first query row of the tile inside the entry), each tile
@@ -451,7 +463,7 @@ extern "C" int llm_wide_attention_prefill(
     if (rc != LLM_OK) return rc;
     if (n_tiles > 65535) return LLM_REFUSED_SIZE;
     if (out_stride % 2 || out_off % 2 || (reinterpret_cast<uintptr_t>(out) & 3u)) return LLM_REFUSED_ALIGN;
-    const size_t smem = (static_cast<size_t>(WP_BM + 2 * WP_BN) * wide_row(dk) + 2 * WP_BN * static_cast<size_t>(wide_row(dv))) * sizeof(bf16);
+    const size_t smem = (static_cast<size_t>(WP_BM + 2 * WP_BN) * wide_row(dk) + 2 * WP_BN * static_cast<size_t>(wide_dv(dv) + 8)) * sizeof(bf16);
     const WideCache c = {static_cast<const bf16*>(keys), static_cast<const bf16*>(values), key_page, value_page, dk, dv, page_size, num_pages};
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define LAUNCH(DD)                                                                                                         \
@@ -463,7 +475,7 @@ extern "C" int llm_wide_attention_prefill(
                    tiles, entry_slot, entry_q_start, entry_q_len, entry_kv_len, block_table, table_stride, nq, nkv, window, \
                    scale * 1.4426950408889634f, status, out_scale, out_stride, out_off);                                   \
     } while (0)
-    WIDE_BY_DV(LAUNCH);
+    WIDE_BY_DV(LAUNCH)
 #undef LAUNCH
     return launch_status();
 }
@@ -485,7 +497,7 @@ extern "C" int llm_wide_attention_decode(
     const int rc = wide_check(q, keys, values, key_page, value_page, nq, nkv, dk, dv, page_size);
     if (rc != LLM_OK) return rc;
     if (num_splits < 1 || num_splits > 65535 || nkv > 65535 || n_rows > 65535 || (num_splits > 1 && !scratch)) return LLM_REFUSED_SIZE;
-    const size_t smem = (static_cast<size_t>(16 + WD_STAGES * WD_BN) * wide_row(dk) + static_cast<size_t>(WD_STAGES * WD_BN) * wide_row(dv)) * sizeof(bf16);
+    const size_t smem = (static_cast<size_t>(16 + 2 * WD_BN) * wide_row(dk) + static_cast<size_t>(2 * WD_BN) * (wide_dv(dv) + 8)) * sizeof(bf16);
     const WideCache c = {static_cast<const bf16*>(keys), static_cast<const bf16*>(values), key_page, value_page, dk, dv, page_size, num_pages};
     float* part_acc = scratch;
     float* part_ml = scratch ? scratch + static_cast<size_t>(n_rows) * nq * num_splits * dv : nullptr;
@@ -499,7 +511,7 @@ extern "C" int llm_wide_attention_decode(
                    positions, token_entry, entry_slot, block_table, table_stride, part_acc, part_ml, static_cast<bf16*>(out), nq, nkv, \
                    window, scale * 1.4426950408889634f, num_splits, status, out_scale, out_stride, out_off);               \
     } while (0)
-    WIDE_BY_DV(LAUNCH);
+    WIDE_BY_DV(LAUNCH)
 #undef LAUNCH
     const int done = launch_status();
     if (done != LLM_OK || num_splits == 1) return done;

@@ -224,6 +224,15 @@ extern "C" int llm_rmsnorm_add(float* h, const void* y, int y_dtype, long long y
     return launch_status();
 }
 
+// block_sum with one barrier: every warp adds the warps' sums up itself.  `scratch` (32 floats) serves one call only.
+__device__ __forceinline__ float block_sum_once(float v, float* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    v = warp_sum(v);
+    if (lane == 0) scratch[warp] = v;
+    __syncthreads();
+    return warp_sum(lane < static_cast<int>((blockDim.x + 31) >> 5) ? scratch[lane] : 0.0f);
+}
+
 // The step between two sublayers of a design that norms a sublayer's input AND its output, in 32-bit throughout:
 //     v      = h[row] + n(y[row]) * w_post (+ join[row])        n(a) = a * rsqrt(mean(a^2) + eps)
 //     h[row] = v                                                (with write_h; the stream is float32)
@@ -241,13 +250,14 @@ __global__ void __launch_bounds__(1024) rmsnorm_sandwich_kernel(float* __restric
                                         long long part_stride, const float* __restrict__ w_post, float eps_post,
                                         const float* __restrict__ join, const float* __restrict__ w_pre, float eps_pre,
                                         TO* __restrict__ out, const int32_t* __restrict__ rows, int hidden, int write_h) {
-    __shared__ float scratch[33];
+    __shared__ float scratch[2][32];
     if constexpr (REG) {
         const int i = threadIdx.x * 8;
         const bool mine = i < hidden;
-        float wp[8], wn[8];                             // the weights are the model's: read before the wait
-        if (mine && w_post) load8(w_post + i, wp);
-        if (mine) load8(w_pre + i, wn);
+        // the weights are the model's: on their way before the wait, but in no registers until they are used (more blocks
+        // of a long step fit an SM)
+        if (mine && w_post) asm volatile("prefetch.global.L1 [%0];\n" ::"l"(w_post + i));
+        if (mine) asm volatile("prefetch.global.L1 [%0];\n" ::"l"(w_pre + i));
         pdl_begin();
         const size_t src = rows ? static_cast<size_t>(rows[blockIdx.x]) : blockIdx.x;
         float* hr = h + src * hidden;
@@ -278,17 +288,21 @@ __global__ void __launch_bounds__(1024) rmsnorm_sandwich_kernel(float* __restric
                 float ss = 0.0f;
 #pragma unroll
                 for (int u = 0; u < 8; ++u) ss += a[u] * a[u];
-                inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_post);
+                inv = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / static_cast<float>(hidden) + eps_post);
             }
+            float wp[8] = {1, 1, 1, 1, 1, 1, 1, 1};
+            if (mine && w_post) load8(w_post + i, wp);
 #pragma unroll
-            for (int u = 0; u < 8; ++u) v[u] += w_post ? (mine ? a[u] * inv * wp[u] : 0.0f) : a[u];
+            for (int u = 0; u < 8; ++u) v[u] += a[u] * inv * wp[u];       // a thread without elements holds zeros
         }
         if (write_h && mine) store8(hr + i, v);
         float ss = 0.0f;
 #pragma unroll
         for (int u = 0; u < 8; ++u) ss += v[u] * v[u];
-        const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_pre);
+        const float inv = 1.0f / sqrtf(block_sum_once(ss, scratch[1]) / static_cast<float>(hidden) + eps_pre);
         if (mine) {
+            float wn[8];
+            load8(w_pre + i, wn);
 #pragma unroll
             for (int u = 0; u < 8; ++u) v[u] = v[u] * inv * wn[u];
             store8(out + static_cast<size_t>(blockIdx.x) * hidden + i, v);
@@ -309,7 +323,7 @@ __global__ void __launch_bounds__(1024) rmsnorm_sandwich_kernel(float* __restric
                 row_s[i] = a;
                 ss += a * a;
             }
-            if (w_post) inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_post);
+            if (w_post) inv = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / static_cast<float>(hidden) + eps_post);
         }
         float ss = 0.0f;
         for (int i = threadIdx.x; i < hidden; i += blockDim.x) {       // each thread meets the elements it wrote itself
@@ -320,7 +334,7 @@ __global__ void __launch_bounds__(1024) rmsnorm_sandwich_kernel(float* __restric
             if (write_h) hr[i] = v;
             ss += v * v;
         }
-        inv = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps_pre);
+        inv = 1.0f / sqrtf(block_sum_once(ss, scratch[1]) / static_cast<float>(hidden) + eps_pre);
         TO* orow = out + static_cast<size_t>(blockIdx.x) * hidden;
         for (int i = threadIdx.x; i < hidden; i += blockDim.x) orow[i] = from_f32<TO>(row_s[i] * inv * w_pre[i]);
     }

@@ -6,7 +6,8 @@ all of it and none, frequencies with and without scaling whose wavelengths fall 
 shorter than a page, no multiple of a page and over several, attention without a mask, chunk sizes that differ between
 layers, dense feed-forwards with different limits, routers that choose one, some and all experts, layers without a
 feed-forward, loops over the start, the middle, the end and the whole of the layers, one pass, several passes, no loop,
-embedding scales and residual factors above, below and equal to one.  Weights are drawn so that activations are of order one
+embedding scales and residual factors below and above one (a table that is the output head too would hide the layers behind
+a token's own row if its scale were large in every model).  Weights are drawn so that activations are of order one
 and a lost key, a chunk off by one or a wrong constant moves the logits by far more than rounding.  This file does not
 import the engine.
 """
@@ -50,7 +51,7 @@ def _config(vocab, width, eps, scale, mult, layers, loop=None):
 
 
 # A: a loop over the middle, three passes; grouped heads, values wider than keys; chunks of 9 and 37 with pages of 16
-PUR_A = _config(103, 48, 1e-5, 2.5, 0.7, [
+PUR_A = _config(103, 48, 1e-5, 0.3, 0.7, [
     _layer(_attn(4, 2, 16, 24, 0.3, chunk=37, rot=(500.0, 8), scaling=(3.0, 1.0, 5.0, 60)), _moe(5, 2, 16)),
     _layer(_attn(6, 2, 8, 8, 0.4, chunk=9, rot=(1.0e4, 8)), _dense(56, 0.9)),
     _layer(_attn(3, 3, 24, 8, 0.25, chunk=37, rot=(200.0, 6), scaling=(2.0, 1.0, 2.0, 40)), _moe(4, 1, 24)),
@@ -59,8 +60,8 @@ PUR_A = _config(103, 48, 1e-5, 2.5, 0.7, [
 PUR_A_PAGE = 16
 
 # B: pages of 4, the loop starts with the first layer, widths that are no multiple of 4, no mask, no rotation, every expert
-# chosen, factors of one
-PUR_B = _config(127, 30, 3e-6, 1.0, 1.0, [
+# chosen, a residual factor of one
+PUR_B = _config(127, 30, 3e-6, 0.3, 1.0, [
     _layer(_attn(3, 3, 8, 10, 0.4, chunk=5, rot=(50.0, 4)), _moe(3, 3, 20)),
     _layer(_attn(2, 1, 12, 6, 0.3), _dense(44, 2.2)),
     _layer(_attn(5, 5, 6, 6, 0.5, chunk=4, rot=(30.0, 6), scaling=(4.0, 0.5, 4.0, 25)), None),
@@ -70,7 +71,7 @@ PUR_B_PAGE = 4
 
 # C: longer sequences; heads of 64 with equal key and value widths and of 32 / 48, chunks of 130 and 70, the loop ends with
 # the last layer
-PUR_C = _config(211, 64, 1e-5, 4.0, 0.35, [
+PUR_C = _config(211, 64, 1e-5, 0.6, 0.35, [
     _layer(_attn(4, 2, 64, 64, 0.125, chunk=130, rot=(2.0e4, 32), scaling=(8.0, 1.0, 4.0, 256)), _dense(96, 1.3)),
     _layer(_attn(4, 4, 32, 48, 0.2, chunk=130, rot=(2.0e3, 16)), _moe(9, 3, 32)),
     _layer(_attn(2, 2, 64, 64, 0.2, chunk=70, rot=(300.0, 64), scaling=(2.0, 2.0, 8.0, 100)), _moe(8, 2, 24)),
@@ -79,7 +80,7 @@ PUR_C = _config(211, 64, 1e-5, 4.0, 0.35, [
 PUR_C_PAGE = 16
 
 # D: no loop; odd sizes throughout, single heads, chunks of one, two and three keys
-PUR_D = _config(89, 36, 1e-6, 0.4, 1.5, [
+PUR_D = _config(89, 36, 1e-6, 1.3, 1.5, [
     _layer(_attn(1, 1, 20, 12, 0.4, chunk=3, rot=(100.0, 6), scaling=(5.0, 1.0, 1.5, 30)), _moe(7, 2, 10)),
     _layer(_attn(6, 3, 4, 12, 1.0, chunk=1, rot=(10.0, 4)), _dense(26, 0.4)),
     _layer(_attn(3, 1, 5, 3, 0.5, chunk=2, rot=(10.0, 2)), _dense(22, 5.0)),
@@ -89,7 +90,7 @@ PUR_D_PAGE = 8
 
 # E: heads of 128 in groups of two, four and one, heads of 96 / 160, the loop over all layers; more experts than a short step
 # has choices
-PUR_E = _config(113, 64, 1e-5, 3.0, 0.5, [
+PUR_E = _config(113, 64, 1e-5, 0.8, 0.5, [
     _layer(_attn(4, 2, 128, 128, 0.09, chunk=140, rot=(1.0e4, 64), scaling=(4.0, 1.0, 4.0, 128)), _moe(12, 2, 40)),
     _layer(_attn(4, 1, 96, 160, 0.1, chunk=33, rot=(1.0e4, 96)), _dense(80, 1.1)),
     _layer(_attn(2, 2, 128, 128, 0.08, chunk=64, rot=(1.0e4, 128)), None),

@@ -24,7 +24,7 @@ def test_plan_of_a_configuration():
     assert isinstance(cfg, PurivikConfig) and cfg.to_dict() == pm.PUR_A
     plan = cfg.plan()
     assert [(s.block, s.starts_pass) for s in plan.order] == [(0, None), (1, 0), (2, None), (1, 1), (2, None), (1, 2), (2, None), (3, None)]
-    assert plan.rejoin == RejoinSpec(3, kind="add") and plan.embedding_scale == 2.5 and plan.tie_word_embeddings
+    assert plan.rejoin == RejoinSpec(3, kind="add") and plan.embedding_scale == 0.3 and plan.tie_word_embeddings
     assert plan.final_norm == NormSpec("rmsnorm", 1e-5, "")
     assert all(b.arrangement == "sandwich_norm" and b.branch_scale == 0.7 and b.layer_scale_names == ("ls1", "ls2") for b in plan.blocks)
     a = plan.blocks[0].mixer

@@ -20,7 +20,7 @@ CASES = {"A": (pm.PUR_A, pm.PUR_A_PAGE, 3), "B": (pm.PUR_B, pm.PUR_B_PAGE, 5), "
          "D": (pm.PUR_D, pm.PUR_D_PAGE, 11), "E": (pm.PUR_E, pm.PUR_E_PAGE, 13)}
 # root mean square over the vocabulary of (difference minus its mean), as a fraction of the reference logits'
 # spread; the float32 run is measured against the plain code in double precision
-LIMIT = {"float32": 1e-4, "bfloat16": 0.12}
+LIMIT = {"float32": 1e-4, "bfloat16": 0.06}
 
 
 def model_of(case):
@@ -66,7 +66,7 @@ def assert_close(got, ref, dtype, what):
         err, limit = ref.error(got[(r, pos)], r, pos), ref.limit(r, pos)
         if err > limit:
             over.append(f"{what}: request {r} position {pos}: {err:.3e} > {limit:.1e}")
-        held += limit <= 2 * LIMIT[dtype]
+        held += limit <= 4 * LIMIT[dtype]
     allowed = 0 if dtype == "float32" else max(1, int(0.03 * len(got)))
     assert len(over) <= allowed, "; ".join(over[:5])
     assert held >= 0.6 * len(got), "too few positions are well conditioned for this to be a test"
