@@ -5,7 +5,7 @@
 //                    equal groups of neighbours; a group's score is the sum of its two largest scores (of
 //                    its one score when a group is one expert) and only experts of the `keep` best groups
 //                    may be chosen (groups = 0: no such limit).  The `top` largest allowed scores are
-//                    chosen (ties go to the lower index); their weights are s / (sum of the chosen s +
+//                    chosen (by their logits where nothing but the scores decides; ties go to the lower index); their weights are s / (sum of the chosen s +
 //                    1e-20) * route_scale.  Written as a dense row of float32 weights [experts] (zero for
 //                    experts that were not chosen) and, optionally, as the lists ids [top], weights [top].
 //                    `softmax` 1: the scores are softmax(z) over all router outputs instead.  `correction`
@@ -60,6 +60,8 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
         for (int i = tid; i < nt * W; i += blockDim.x) xs[i] = to_f32(x[t0 * W + i]);
     }
     __syncthreads();
+    // a plain choice by sigmoid scores is made by the logits, which order alike and do not crowd together near one
+    const bool by_logit = !softmax && !correction && groups == 0;
     const int rows = E + (shared_w ? 1 : 0);
     for (int e = warp; e < rows; e += MOE_ROUTE_THREADS / 32) {    // a warp an expert: its row against the block's tokens
         const float* w = e < E ? wr + static_cast<size_t>(e) * W : shared_w;
@@ -91,7 +93,7 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
                 continue;
             }
             if (bias) d += bias[e];
-            if (lane == 0 && k < nt) score[k * E + e] = softmax ? d : 1.0f / (1.0f + expf(-d));
+            if (lane == 0 && k < nt) score[k * E + e] = softmax || by_logit ? d : 1.0f / (1.0f + expf(-d));
         }
     }
     __syncthreads();
@@ -153,6 +155,7 @@ __global__ void moe_route_kernel(const TX* __restrict__ x, const float* __restri
             chosen[n] = best;
             if (best >= 0) {
                 ok[best] = 0;
+                if (by_logit) sc[best] = 1.0f / (1.0f + expf(-sc[best]));       // chosen once: from here on its score
                 total += sc[best];
             }
         }

@@ -546,6 +546,12 @@ def test_router_scores_are_the_weights(E, top, W):
     for t in range(T):
         mine = {int(e): float(a) for e, a in zip(ids[t].tolist(), wts[t].tolist())}
         assert set(mine) == set(pick[t].tolist()) and all(abs(mine[e] - float(want[t, e])) < 1e-6 for e in mine)
+    # scores that crowd together just below one: the choice is still the largest
+    hot = {"router": w["router"] * 0 + 1.0 / W}
+    hot["router"] = hot["router"] * (17.0 + torch.arange(E, dtype=F64)[:, None] / 64)
+    ones = torch.ones(T, W, dtype=F64)
+    _, ids, _ = ops.moe_route(_f32(ones), _f32(hot["router"]), top, None, 1.0, lists=True, normalize=False)
+    assert ids.tolist() == [list(range(E - 1, E - 1 - top, -1))] * T
     shares = ops.moe_route(_f32(x), _f32(w["router"]), top, None, 1.0)
     assert (shares.double().cpu() - want / want.sum(1, keepdim=True)).abs().max() < 1e-6
     assert (shares.double().cpu() - want).abs().max() > 0.05
