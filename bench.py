@@ -1025,7 +1025,7 @@ def purivik_bench(args, pk, measure) -> int:
             flops=flops(span, d, d))
     add(f"prompt attention, mma, a window of {chunk} with a sink and kept keys (like: Vugedra's): {T} tokens",
         lambda: ops.paged_attention_prefill_biased(qa, oa, 0, cache, *entry, d, PAGE, chunk, d ** -0.5, status, keep_first=4, sink=sinks), flops=flops(chunk, d, d))
-    for dk, dv in ((64, 80), (128, 192), (128, 128), (256, 256)):
+    for dk, dv in ((64, 96), (128, 192), (128, 128), (256, 256)):
         keys, values = bf(pages, kv, PAGE, dk), bf(pages, kv, PAGE, dv)
         q, o = bf(T, heads * dk), torch.empty(T, heads * dv, device=dev, dtype=torch.bfloat16)
         add(f"prompt attention, keys of {dk}, values of {dv}, chunks of {chunk} (new): {T} tokens",
@@ -1046,7 +1046,7 @@ def purivik_bench(args, pk, measure) -> int:
         add(f"decode attention, {label}: {Bd} tokens at position {ctx - 1}",
             lambda span=span: ops.paged_attention_decode(qa[:Bd], oa[:Bd], dcache, *step, d, PAGE, span, d ** -0.5, 1, status), nbytes=kv_bytes(d, d))
     del dcache
-    for dk, dv in ((64, 80), (128, 192), (128, 128)):
+    for dk, dv in ((64, 96), (128, 192), (128, 128)):
         keys, values = bf(Bd * dpages, kv, PAGE, dk), bf(Bd * dpages, kv, PAGE, dv)
         q, o = bf(Bd, heads * dk), torch.empty(Bd, heads * dv, device=dev, dtype=torch.bfloat16)
         for splits in (1, 2):

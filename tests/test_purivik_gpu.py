@@ -440,7 +440,7 @@ def test_tensor_core_attention_within_chunks(d, group, chunk):
         assert (plain(other) - ref).abs().max() > 0.3
 
 
-@pytest.mark.parametrize("H,G,D,V,span,page", [(4, 4, 64, 80, -120, 16), (6, 2, 32, 48, -30, 16), (16, 1, 128, 256, -300, 64), (3, 3, 256, 128, 100, 16),
+@pytest.mark.parametrize("H,G,D,V,span,page", [(6, 3, 64, 88, -110, 16), (6, 2, 32, 48, -30, 16), (16, 1, 128, 256, -300, 64), (3, 3, 256, 128, 100, 16),
                                                (8, 2, 8, 8, None, 4), (2, 1, 72, 24, -1, 8), (4, 2, 256, 256, -64, 16), (5, 5, 96, 96, 65, 5),
                                                (4, 2, 40, 192, -128, 16)])
 def test_tensor_core_attention_of_any_widths(H, G, D, V, span, page):
